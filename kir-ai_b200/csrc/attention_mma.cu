@@ -54,6 +54,11 @@ __device__ __forceinline__ uint32_t tile_offset(int row, int chunk) {
     return (uint32_t)((chunk >> 3) * (ROWS * 128) + row * 128 + (((chunk & 7) ^ (row & 7)) << 4));
 }
 
+// A merged row's value: the weighted sum over the weights' sum (and a sink's weight, see softmax_inverse).
+__device__ __forceinline__ float softmax_value(float acc, float m, float sum, const float* sinks, int head) {
+    return sinks ? acc * softmax_inverse(m, sum, sinks, head) : (sum > 0.0f ? acc / sum : 0.0f);
+}
+
 // Running softmax state of the two rows (g and g + 8) that a thread of an m16 tile holds.
 template <int D>
 struct WarpState {
@@ -431,8 +436,8 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap kv_map, const bf16*
         l += __shfl_xor_sync(0xffffffffu, l, 2);
         const int row = row0 + warp * 16 + (lane >> 2) + r * 8;
         if (row >= rows_total) continue;
-        const float inv = l > 0.0f ? 1.0f / l : 0.0f;
         const int token = row / group, head = kv_head * group + row % group;
+        const float inv = softmax_inverse(st.m[r], l, form.sinks, head);
         bf16* dst = out + ((size_t)(q_begin + token) * q_heads + head) * head_dim;
 #pragma unroll
         for (int n = 0; n < D / 8; ++n) {
@@ -985,7 +990,8 @@ __device__ __forceinline__ int decode_attend_range(const CUtensorMap& kv_map, co
             l_all += src[D + 1] * weight;
         }
         if (dst_partial == nullptr) {
-            out[((size_t)req * q_heads + kv_head * group + row) * head_dim + col] = from_f32<bf16>(l_all > 0.0f ? acc / l_all : 0.0f);
+            const int head = kv_head * group + row;
+            out[((size_t)req * q_heads + head) * head_dim + col] = from_f32<bf16>(softmax_value(acc, m_all, l_all, form.sinks, head));
         } else {
             float* dst = dst_partial + (size_t)row * partial_stride;
             dst[col] = acc;
@@ -1079,7 +1085,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap kv_map, DecodeArgs a
                     acc += src[col] * weight;
                     l_all += src[head_dim + 1] * weight;
                 }
-                out[((size_t)req * args.q_heads + kv_head * group + row) * head_dim + col] = from_f32<bf16>(l_all > 0.0f ? acc / l_all : 0.0f);
+                const int head = kv_head * group + row;
+                out[((size_t)req * args.q_heads + head) * head_dim + col] = from_f32<bf16>(softmax_value(acc, m_all, l_all, args.form.sinks, head));
             }
         }
         decode_stamp(args, 4);
@@ -1195,7 +1202,7 @@ attention_decode_balanced_kernel(const __grid_constant__ CUtensorMap kv_map, Dec
 __global__ void __launch_bounds__(128)
 attention_merge_balanced_kernel(const float* __restrict__ partial, bf16* __restrict__ out,
                                 const int* __restrict__ context_len, int requests, int q_heads, int kv_heads,
-                                int head_dim, int window, int tile_keys, int ctas) {
+                                int head_dim, int window, int tile_keys, int ctas, const float* __restrict__ sinks) {
     pdl_launch_dependents();
     __shared__ int prefix[DECODE_MAX_REQUESTS + 1];
     __shared__ float warp_max[4];
@@ -1234,12 +1241,12 @@ attention_merge_balanced_kernel(const float* __restrict__ partial, bf16* __restr
             acc += src[col] * weight;
             l_all += src[head_dim + 1] * weight;
         }
-        dst[col] = from_f32<bf16>(l_all > 0.0f ? acc / l_all : 0.0f);
+        dst[col] = from_f32<bf16>(softmax_value(acc, m_all, l_all, sinks, head));
     }
 }
 
 __global__ void attention_merge_splits_kernel(const float* __restrict__ partial, bf16* __restrict__ out, int head_dim,
-                                              int num_splits) {
+                                              int num_splits, int q_heads, const float* __restrict__ sinks) {
     pdl_launch_dependents();
     pdl_wait();
     // one block per (request, head); the splits are read eight at a time, so that their loads are in flight together
@@ -1273,7 +1280,7 @@ __global__ void attention_merge_splits_kernel(const float* __restrict__ partial,
                 l_all += l[u] * weight;
             }
         }
-        out[rh * head_dim + col] = from_f32<bf16>(l_all > 0.0f ? acc / l_all : 0.0f);
+        out[rh * head_dim + col] = from_f32<bf16>(softmax_value(acc, m_all, l_all, sinks, (int)(rh % q_heads)));
     }
 }
 
@@ -1293,7 +1300,7 @@ template <int D>
 int prefill_launch(const void* q, const void* cache, void* out, const int* block_table, const int* query_start,
                    const int* context_len, int requests, int max_query_len, int q_heads, int kv_heads, int head_dim,
                    long q_row_stride, int page_size, int table_width, int num_pages, int window, float scale,
-                   int* error_flag, cudaStream_t stream, float softcap = 0.0f) {
+                   int* error_flag, cudaStream_t stream, float softcap = 0.0f, const float* sinks = nullptr) {
     using Smem = PrefillSmem<D>;
     const int group = q_heads / kv_heads;
     const int box_rows = page_size < PF_BN ? page_size : PF_BN;
@@ -1308,14 +1315,15 @@ int prefill_launch(const void* q, const void* cache, void* out, const int* block
     if (grid.y > 65535) return KIRAI_ERR_BAD_SIZE;
     return launch_pdl(kernel, grid, dim3((PF_WARPS + 1) * 32), (size_t)Smem::total, stream, 1u, kv_map, (const bf16*)q,
                       (bf16*)out, block_table, query_start, context_len, q_heads, kv_heads, head_dim, q_row_stride,
-                      page_size, box_rows, table_width, num_pages, window, make_score_form(scale, softcap), error_flag);
+                      page_size, box_rows, table_width, num_pages, window, make_score_form(scale, softcap, sinks), error_flag);
 }
 
 template <int D>
 int decode_launch(const void* q, const void* cache, void* out, float* partial, const int* block_table,
                   const int* context_len, int requests, int q_heads, int kv_heads, int head_dim, long q_row_stride,
                   int page_size, int table_width, int num_pages, int window, float scale, int num_splits,
-                  int* error_flag, cudaStream_t stream, const FuseQK* fuse = nullptr, float softcap = 0.0f) {
+                  int* error_flag, cudaStream_t stream, const FuseQK* fuse = nullptr, float softcap = 0.0f,
+                  const float* sinks = nullptr) {
     using Smem = DecodeSmem<D>;
     const int box_rows = page_size < Smem::BN ? page_size : Smem::BN;
     if (Smem::BN % box_rows != 0 || page_size % box_rows != 0) return KIRAI_ERR_UNSUPPORTED;  // page sizes: powers of two
@@ -1332,7 +1340,7 @@ int decode_launch(const void* q, const void* cache, void* out, float* partial, c
     if (err != cudaSuccess) return (int)err;
     if (fuse && head_dim != D) return KIRAI_ERR_UNSUPPORTED;  // the fused preparation works on whole heads of 64, 128 or 256
     DecodeArgs args{(const bf16*)q, block_table, q_heads, kv_heads, head_dim, q_row_stride, page_size, box_rows,
-                    table_width, num_pages, window, make_score_form(scale, softcap), error_flag};
+                    table_width, num_pages, window, make_score_form(scale, softcap, sinks), error_flag};
     if (fuse) {
         args.fuse = 1, args.q_weight = fuse->q_weight, args.k_weight = fuse->k_weight, args.inv_freq = fuse->inv_freq;
         args.eps = fuse->eps, args.cache = (bf16*)const_cast<void*>(cache);
@@ -1347,14 +1355,15 @@ int decode_launch(const void* q, const void* cache, void* out, float* partial, c
                             (bf16*)out, partial, context_len, num_splits);
     if (status || num_splits == 1) return status;
     return launch_pdl(attention_merge_splits_kernel, dim3(requests * q_heads), dim3(128), 0, stream, 1u,
-                      (const float*)partial, (bf16*)out, head_dim, num_splits);
+                      (const float*)partial, (bf16*)out, head_dim, num_splits, q_heads, sinks);
 }
 
 template <int D>
 int decode_balanced_launch(const void* q, const void* cache, void* out, float* partial, const int* block_table,
                            const int* context_len, int requests, int q_heads, int kv_heads, int head_dim,
                            long q_row_stride, int page_size, int table_width, int num_pages, int window, float scale,
-                           int ctas, int* error_flag, cudaStream_t stream, const FuseQK* fuse = nullptr, float softcap = 0.0f) {
+                           int ctas, int* error_flag, cudaStream_t stream, const FuseQK* fuse = nullptr, float softcap = 0.0f,
+                  const float* sinks = nullptr) {
     using Smem = DecodeSmem<D>;
     const int box_rows = page_size < Smem::BN ? page_size : Smem::BN;
     if (Smem::BN % box_rows != 0 || page_size % box_rows != 0) return KIRAI_ERR_UNSUPPORTED;  // page sizes: powers of two
@@ -1366,7 +1375,7 @@ int decode_balanced_launch(const void* q, const void* cache, void* out, float* p
     if (err != cudaSuccess) return (int)err;
     if (fuse && head_dim != D) return KIRAI_ERR_UNSUPPORTED;  // the fused preparation works on whole heads of 64, 128 or 256
     DecodeArgs args{(const bf16*)q, block_table, q_heads, kv_heads, head_dim, q_row_stride, page_size, box_rows,
-                    table_width, num_pages, window, make_score_form(scale, softcap), error_flag};
+                    table_width, num_pages, window, make_score_form(scale, softcap, sinks), error_flag};
     if (fuse) {
         args.fuse = 1, args.q_weight = fuse->q_weight, args.k_weight = fuse->k_weight, args.inv_freq = fuse->inv_freq;
         args.eps = fuse->eps, args.cache = (bf16*)const_cast<void*>(cache);
@@ -1376,7 +1385,7 @@ int decode_balanced_launch(const void* q, const void* cache, void* out, float* p
     if (status) return status;
     return launch_pdl(attention_merge_balanced_kernel, dim3(requests * q_heads), dim3(128), 0, stream, 1u,
                       (const float*)partial, (bf16*)out, context_len, requests, q_heads, kv_heads, head_dim, window,
-                      (int)Smem::BN, ctas);
+                      (int)Smem::BN, ctas, sinks);
 }
 
 int check_common(int q_heads, int kv_heads, int head_dim, long q_row_stride, const void* q) {
@@ -1396,7 +1405,8 @@ static int attention_prefill_entry(const void* q, const void* cache, void* out, 
                                    const int* query_start, const int* context_len, int requests,
                                    int max_query_len, int q_heads, int kv_heads, int head_dim,
                                    long q_row_stride, int page_size, int table_width, int num_pages,
-                                   int window, float scale, float softcap, int* error_flag, cudaStream_t stream) {
+                                   int window, float scale, float softcap, int* error_flag, cudaStream_t stream,
+                                   const float* sinks = nullptr) {
     if (requests <= 0 || max_query_len <= 0) return 0;
     int bad = check_common(q_heads, kv_heads, head_dim, q_row_stride, q);
     if (bad) return bad;
@@ -1404,7 +1414,7 @@ static int attention_prefill_entry(const void* q, const void* cache, void* out, 
 #define KIRAI_PF(D) \
     return prefill_launch<D>(q, cache, out, block_table, query_start, context_len, requests, max_query_len, q_heads, \
                              kv_heads, head_dim, q_row_stride, page_size, table_width, num_pages, window, scale, \
-                             error_flag, stream, softcap)
+                             error_flag, stream, softcap, sinks)
     if (head_dim <= 64) KIRAI_PF(64);
     if (head_dim <= 128) KIRAI_PF(128);
     KIRAI_PF(256);
@@ -1474,7 +1484,7 @@ static int attention_decode_entry(const void* q, const void* cache, void* out, f
                                   const int* block_table, const int* context_len, int requests,
                                   int q_heads, int kv_heads, int head_dim, long q_row_stride, int page_size,
                                   int table_width, int num_pages, int window, float scale, float softcap, int num_splits,
-                                  int* error_flag, cudaStream_t stream) {
+                                  int* error_flag, cudaStream_t stream, const float* sinks = nullptr) {
     if (requests <= 0) return 0;
     int bad = check_common(q_heads, kv_heads, head_dim, q_row_stride, q);
     if (bad) return bad;
@@ -1484,7 +1494,7 @@ static int attention_decode_entry(const void* q, const void* cache, void* out, f
 #define KIRAI_DC(D) \
     return decode_launch<D>(q, cache, out, partial, block_table, context_len, requests, q_heads, kv_heads, head_dim, \
                             q_row_stride, page_size, table_width, num_pages, window, scale, num_splits, error_flag, \
-                            stream, nullptr, softcap)
+                            stream, nullptr, softcap, sinks)
     if (head_dim <= 64) KIRAI_DC(64);
     if (head_dim <= 128) KIRAI_DC(128);
     KIRAI_DC(256);
@@ -1518,7 +1528,8 @@ static int attention_decode_balanced_entry(const void* q, const void* cache, voi
                                            const int* block_table, const int* context_len, int requests,
                                            int q_heads, int kv_heads, int head_dim, long q_row_stride,
                                            int page_size, int table_width, int num_pages, int window,
-                                           float scale, float softcap, int ctas, int* error_flag, cudaStream_t stream) {
+                                           float scale, float softcap, int ctas, int* error_flag, cudaStream_t stream,
+                                           const float* sinks = nullptr) {
     if (requests <= 0) return 0;
     int bad = check_common(q_heads, kv_heads, head_dim, q_row_stride, q);
     if (bad) return bad;
@@ -1528,7 +1539,7 @@ static int attention_decode_balanced_entry(const void* q, const void* cache, voi
 #define KIRAI_DCB(D) \
     return decode_balanced_launch<D>(q, cache, out, partial, block_table, context_len, requests, q_heads, kv_heads, \
                                      head_dim, q_row_stride, page_size, table_width, num_pages, window, scale, ctas, \
-                                     error_flag, stream, nullptr, softcap)
+                                     error_flag, stream, nullptr, softcap, sinks)
     if (head_dim <= 64) KIRAI_DCB(64);
     if (head_dim <= 128) KIRAI_DCB(128);
     KIRAI_DCB(256);
@@ -1555,6 +1566,38 @@ KIRAI_EXPORT int kirai_attention_decode_balanced_softcap_bf16(const void* q, con
     return attention_decode_balanced_entry(q, cache, out, partial, block_table, context_len, requests, q_heads, kv_heads,
                                            head_dim, q_row_stride, page_size, table_width, num_pages, window, scale, softcap,
                                            ctas, error_flag, stream);
+}
+
+// The three entry points above with a sink per query head beside the visible keys (`sinks` [q_heads] float32, see
+// ScoreForm); it is taken into a row's sum once, where the row's ranges are together.
+KIRAI_EXPORT int kirai_attention_prefill_sink_bf16(const void* q, const void* cache, void* out, const int* block_table,
+                                                   const int* query_start, const int* context_len, int requests,
+                                                   int max_query_len, int q_heads, int kv_heads, int head_dim,
+                                                   long q_row_stride, int page_size, int table_width, int num_pages,
+                                                   int window, float scale, float softcap, const float* sinks,
+                                                   int* error_flag, cudaStream_t stream) {
+    return attention_prefill_entry(q, cache, out, block_table, query_start, context_len, requests, max_query_len, q_heads,
+                                   kv_heads, head_dim, q_row_stride, page_size, table_width, num_pages, window, scale,
+                                   softcap, error_flag, stream, sinks);
+}
+KIRAI_EXPORT int kirai_attention_decode_sink_bf16(const void* q, const void* cache, void* out, float* partial,
+                                                  const int* block_table, const int* context_len, int requests,
+                                                  int q_heads, int kv_heads, int head_dim, long q_row_stride, int page_size,
+                                                  int table_width, int num_pages, int window, float scale, float softcap,
+                                                  const float* sinks, int num_splits, int* error_flag, cudaStream_t stream) {
+    return attention_decode_entry(q, cache, out, partial, block_table, context_len, requests, q_heads, kv_heads, head_dim,
+                                  q_row_stride, page_size, table_width, num_pages, window, scale, softcap, num_splits,
+                                  error_flag, stream, sinks);
+}
+KIRAI_EXPORT int kirai_attention_decode_balanced_sink_bf16(const void* q, const void* cache, void* out, float* partial,
+                                                           const int* block_table, const int* context_len, int requests,
+                                                           int q_heads, int kv_heads, int head_dim, long q_row_stride,
+                                                           int page_size, int table_width, int num_pages, int window,
+                                                           float scale, float softcap, const float* sinks, int ctas,
+                                                           int* error_flag, cudaStream_t stream) {
+    return attention_decode_balanced_entry(q, cache, out, partial, block_table, context_len, requests, q_heads, kv_heads,
+                                           head_dim, q_row_stride, page_size, table_width, num_pages, window, scale, softcap,
+                                           ctas, error_flag, stream, sinks);
 }
 
 // The two decode entry points with the preparation of queries and keys inside: `qkv` holds the rows that the q, k, v

@@ -21,7 +21,7 @@ paged_attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ cach
                              const int* __restrict__ block_table, const int* __restrict__ request_of_token,
                              const int* __restrict__ positions, int q_heads, int kv_heads, int head_dim,
                              long q_row_stride, int page_size, int table_width, int num_pages, int window, float scale,
-                             float softcap, int* __restrict__ error_flag) {
+                             float softcap, const float* __restrict__ sinks, int* __restrict__ error_flag) {
     extern __shared__ float smem[];
     float* q_s = smem;                       // [head_dim]
     float* o_s = smem + head_dim;            // [ATT_WARPS][head_dim]
@@ -92,12 +92,14 @@ paged_attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ cach
         weight[w] = (m_s[w] == -INFINITY) ? 0.0f : expf(m_s[w] - m_all);
         l_all += l_s[w] * weight[w];
     }
+    // (softmax_inverse works with base-2 exponents)
+    const float inverse = softmax_inverse(m_all * 1.4426950408889634f, l_all, sinks, head);
     T* out_row = out + ((size_t)token * q_heads + head) * head_dim;
     for (int i = threadIdx.x; i < head_dim; i += blockDim.x) {
         float acc = 0.0f;
 #pragma unroll
         for (int w = 0; w < ATT_WARPS; ++w) acc += o_s[w * head_dim + i] * weight[w];
-        out_row[i] = from_f32<T>(l_all > 0.0f ? acc / l_all : 0.0f);
+        out_row[i] = from_f32<T>(sinks ? acc * inverse : (l_all > 0.0f ? acc / l_all : 0.0f));
     }
 }
 
@@ -105,7 +107,8 @@ template <typename T>
 static int paged_attention_plain_launch(const void* q, const void* cache, void* out, const int* block_table,
                                         const int* request_of_token, const int* positions, int tokens, int q_heads,
                                         int kv_heads, int head_dim, long q_row_stride, int page_size, int table_width,
-                                        int num_pages, int window, float scale, float softcap, int* error_flag, cudaStream_t stream) {
+                                        int num_pages, int window, float scale, float softcap, int* error_flag, cudaStream_t stream,
+                                        const float* sinks = nullptr) {
     if (tokens <= 0) return 0;
     if (head_dim > 32 * ATT_MAX_PER_LANE || head_dim <= 0) return KIRAI_ERR_BAD_SIZE;
     if (kv_heads <= 0 || q_heads % kv_heads != 0) return KIRAI_ERR_BAD_SIZE;
@@ -114,7 +117,7 @@ static int paged_attention_plain_launch(const void* q, const void* cache, void* 
     dim3 grid(tokens, q_heads);
     paged_attention_plain_kernel<T><<<grid, ATT_WARPS * 32, smem, stream>>>(
         (const T*)q, (const T*)cache, (T*)out, block_table, request_of_token, positions, q_heads, kv_heads, head_dim,
-        q_row_stride, page_size, table_width, num_pages, window, scale, softcap, error_flag);
+        q_row_stride, page_size, table_width, num_pages, window, scale, softcap, sinks, error_flag);
     return launch_status();
 }
 
@@ -156,4 +159,26 @@ KIRAI_EXPORT int kirai_paged_attention_plain_softcap_bf16(const void* q, const v
     return paged_attention_plain_launch<bf16>(q, cache, out, block_table, request_of_token, positions, tokens, q_heads,
                                               kv_heads, head_dim, q_row_stride, page_size, table_width, num_pages,
                                               window, scale, softcap, error_flag, stream);
+}
+
+// The same with a sink per query head beside the visible keys (`sinks` [q_heads] float32, see ScoreForm).
+KIRAI_EXPORT int kirai_paged_attention_plain_sink_f32(const void* q, const void* cache, void* out, const int* block_table,
+                                                      const int* request_of_token, const int* positions, int tokens,
+                                                      int q_heads, int kv_heads, int head_dim, long q_row_stride,
+                                                      int page_size, int table_width, int num_pages, int window,
+                                                      float scale, float softcap, const float* sinks, int* error_flag,
+                                                      cudaStream_t stream) {
+    return paged_attention_plain_launch<float>(q, cache, out, block_table, request_of_token, positions, tokens, q_heads,
+                                               kv_heads, head_dim, q_row_stride, page_size, table_width, num_pages,
+                                               window, scale, softcap, error_flag, stream, sinks);
+}
+KIRAI_EXPORT int kirai_paged_attention_plain_sink_bf16(const void* q, const void* cache, void* out, const int* block_table,
+                                                       const int* request_of_token, const int* positions, int tokens,
+                                                       int q_heads, int kv_heads, int head_dim, long q_row_stride,
+                                                       int page_size, int table_width, int num_pages, int window,
+                                                       float scale, float softcap, const float* sinks, int* error_flag,
+                                                       cudaStream_t stream) {
+    return paged_attention_plain_launch<bf16>(q, cache, out, block_table, request_of_token, positions, tokens, q_heads,
+                                              kv_heads, head_dim, q_row_stride, page_size, table_width, num_pages,
+                                              window, scale, softcap, error_flag, stream, sinks);
 }

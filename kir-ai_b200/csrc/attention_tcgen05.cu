@@ -472,7 +472,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const bf
         if (ok) ok = mbar_wait_hot(smem_addr(o_ready), (uint32_t)(num_tiles - 1) & 1u);
         tc_fence_after();
         if (ok) {
-            const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+            const float inv = softmax_inverse(m_used, l, valid ? form.sinks : nullptr, kv_head * group + row % group);
             bf16* dst = nullptr;
             if (valid) {
                 const int token = row / group, head = kv_head * group + row % group;
@@ -513,7 +513,7 @@ template <int D>
 int launch(const void* q, const void* cache, void* out, const int* block_table, const int* query_start,
            const int* context_len, int requests, int max_query_len, int q_heads, int kv_heads, int head_dim,
            long q_row_stride, int page_size, int table_width, int num_pages, int window, float scale, float softcap,
-           int* error_flag, cudaStream_t stream) {
+           int* error_flag, cudaStream_t stream, const float* sinks) {
     using Smem = TcAttnSmem<D>;
     const int group = q_heads / kv_heads;
     const int box_rows = page_size < TA_BN ? page_size : TA_BN;
@@ -533,7 +533,7 @@ int launch(const void* q, const void* cache, void* out, const int* block_table, 
     if (grid.y > 65535) return KIRAI_ERR_BAD_SIZE;
     return launch_pdl(kernel, grid, dim3(TA_THREADS), (size_t)Smem::total, stream, 1u, kv_map, (const bf16*)q, (bf16*)out,
                       block_table, query_start, context_len, q_heads, kv_heads, head_dim, q_row_stride, page_size, box_rows,
-                      piece_rows, table_width, num_pages, window, make_score_form(scale, softcap), error_flag);
+                      piece_rows, table_width, num_pages, window, make_score_form(scale, softcap, sinks), error_flag);
 }
 
 }  // namespace
@@ -544,7 +544,8 @@ static int attention_prefill_tc_entry(const void* q, const void* cache, void* ou
                                       const int* query_start, const int* context_len, int requests,
                                       int max_query_len, int q_heads, int kv_heads, int head_dim,
                                       long q_row_stride, int page_size, int table_width, int num_pages,
-                                      int window, float scale, float softcap, int* error_flag, cudaStream_t stream) {
+                                      int window, float scale, float softcap, int* error_flag, cudaStream_t stream,
+                                      const float* sinks = nullptr) {
     if (requests <= 0 || max_query_len <= 0) return 0;
     if (kv_heads <= 0 || q_heads % kv_heads != 0) return KIRAI_ERR_BAD_SIZE;
     const int group = q_heads / kv_heads;
@@ -554,12 +555,12 @@ static int attention_prefill_tc_entry(const void* q, const void* cache, void* ou
     if (requests > 65535 || kv_heads > 65535) return KIRAI_ERR_BAD_SIZE;
     if (head_dim <= 64)
         return launch<64>(q, cache, out, block_table, query_start, context_len, requests, max_query_len, q_heads, kv_heads,
-                          head_dim, q_row_stride, page_size, table_width, num_pages, window, scale, softcap, error_flag, stream);
+                          head_dim, q_row_stride, page_size, table_width, num_pages, window, scale, softcap, error_flag, stream, sinks);
     if (head_dim <= 128)
         return launch<128>(q, cache, out, block_table, query_start, context_len, requests, max_query_len, q_heads, kv_heads,
-                           head_dim, q_row_stride, page_size, table_width, num_pages, window, scale, softcap, error_flag, stream);
+                           head_dim, q_row_stride, page_size, table_width, num_pages, window, scale, softcap, error_flag, stream, sinks);
     return launch<256>(q, cache, out, block_table, query_start, context_len, requests, max_query_len, q_heads, kv_heads,
-                       head_dim, q_row_stride, page_size, table_width, num_pages, window, scale, softcap, error_flag, stream);
+                       head_dim, q_row_stride, page_size, table_width, num_pages, window, scale, softcap, error_flag, stream, sinks);
 }
 
 KIRAI_EXPORT int kirai_attention_prefill_tc_bf16(const void* q, const void* cache, void* out, const int* block_table,
@@ -582,4 +583,16 @@ KIRAI_EXPORT int kirai_attention_prefill_tc_softcap_bf16(const void* q, const vo
     return attention_prefill_tc_entry(q, cache, out, block_table, query_start, context_len, requests, max_query_len, q_heads,
                                       kv_heads, head_dim, q_row_stride, page_size, table_width, num_pages, window, scale,
                                       softcap, error_flag, stream);
+}
+
+// The same with a sink per query head beside the visible keys (`sinks` [q_heads] float32, see ScoreForm).
+KIRAI_EXPORT int kirai_attention_prefill_tc_sink_bf16(const void* q, const void* cache, void* out, const int* block_table,
+                                                      const int* query_start, const int* context_len, int requests,
+                                                      int max_query_len, int q_heads, int kv_heads, int head_dim,
+                                                      long q_row_stride, int page_size, int table_width, int num_pages,
+                                                      int window, float scale, float softcap, const float* sinks,
+                                                      int* error_flag, cudaStream_t stream) {
+    return attention_prefill_tc_entry(q, cache, out, block_table, query_start, context_len, requests, max_query_len, q_heads,
+                                      kv_heads, head_dim, q_row_stride, page_size, table_width, num_pages, window, scale,
+                                      softcap, error_flag, stream, sinks);
 }

@@ -27,6 +27,8 @@ SOURCES = [
     "mixer_forms.cu",
     "state_forms.cu",
     "state_chunks.cu",
+    "gated_scan.cu",
+    "stream_forms.cu",
     "experts.cu",
     "gemm_simt.cu",
     "attention_plain.cu",

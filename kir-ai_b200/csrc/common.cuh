@@ -23,6 +23,7 @@
 #define KIRAI_FLAG_NO_PAGE_READ 3
 #define KIRAI_FLAG_WAIT_RAN_OUT 4
 #define KIRAI_FLAG_NO_MAXIMUM 5
+#define KIRAI_FLAG_BAD_POSITION 6
 
 typedef __nv_bfloat16 bf16;
 
@@ -128,12 +129,17 @@ __host__ __device__ __forceinline__ int first_visible_key(int pos, int window) {
 // absolute error stays near 1e-7; large |x| needs no clamp: the exponential gives inf or 0 there, and the reciprocal of
 // inf is 0), and the factors around it are folded on the host: cap_in = 2 log2(e) scale / c, cap_log2 = c log2(e)
 // (0: no cap), cap_out = -2 cap_log2, so that a capped score is a multiply, ex2, an add, rcp and a multiply-add.
+// `sinks` (null: none) holds one number per query head, the score of a key that every query of the head sees beside its
+// visible keys and that has no value: it stands in the softmax's denominator only (0 adds one to the sum of the
+// exponentials).
 struct ScoreForm {
     float scale_log2, cap_in, cap_log2, cap_out;
+    const float* sinks;
 };
 
-static inline ScoreForm make_score_form(float scale, float softcap) {
+static inline ScoreForm make_score_form(float scale, float softcap, const float* sinks = nullptr) {
     ScoreForm form;
+    form.sinks = sinks;
     form.scale_log2 = scale * 1.4426950408889634f;
     form.cap_in = softcap > 0.0f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.0f;
     form.cap_log2 = softcap > 0.0f ? softcap * 1.4426950408889634f : 0.0f;
@@ -146,6 +152,16 @@ __device__ __forceinline__ float capped_exponent(float raw, const ScoreForm& for
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(raw * form.cap_in));
     asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.0f));
     return fmaf(form.cap_out, r, form.cap_log2);
+}
+
+// What an accumulated row of values is multiplied by at the end: 1 / sum, the weights being exp2(score - m) and `sum`
+// their sum; with a sink the sum takes the sink's weight in, on the scale of the greater of the two exponents.
+__device__ __forceinline__ float softmax_inverse(float m, float sum, const float* sinks, int head) {
+    if (!sinks) return sum > 0.0f ? 1.0f / sum : 0.0f;
+    const float s = sinks[head] * 1.4426950408889634f;
+    const float top = fmaxf(m, s);
+    const float keep = m == -INFINITY ? 0.0f : exp2f(m - top);
+    return keep / (sum * keep + exp2f(s - top));
 }
 
 static inline int launch_status() { return (int)cudaGetLastError(); }

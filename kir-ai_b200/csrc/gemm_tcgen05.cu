@@ -1283,7 +1283,8 @@ KIRAI_EXPORT int kirai_gemm_bf16_grouped(const void* A, const void* W, int tiled
 // The one entry point of the tensor-core product, A[M, K] (row stride lda) times W[N, K] transposed.
 //   tiled:  W is in the tiled form described at the top of this file, else row-major.
 //   form 0: C[M, N] bf16.  1: C[M, N] float.  2: C[M, N / 2] = silu(gate) * up, W's rows in groups of 8 gate rows
-//           followed by their 8 up rows.  5: as 2 with the tanh form of gelu in place of silu.  4: C[M, N] bf16 =
+//           followed by their 8 up rows.  5: as 2 with the tanh form of gelu in place of silu.  7: as 2 with the clamped form
+//           (gate_act 2 of Epilogue, gate_limit and gate_slope) in place of silu.  4: C[M, N] bf16 =
 //           relu(product)^2.  3: residual[M, N] (float, in place) += product, C[M, N] =
 //           bf16(residual * norm_weight[n]) and sumsq_out[parts][M] = each column tile's share of sum_n residual^2.
 //   row_sumsq (forms 0-2, may be null): the rows of A were left unscaled by an RMSNorm; row m of the product is
@@ -1292,7 +1293,7 @@ KIRAI_EXPORT int kirai_gemm_bf16_grouped(const void* A, const void* W, int tiled
 KIRAI_EXPORT int kirai_gemm_bf16_general(const void* A, const void* W, int tiled, void* C, int M, int N, int K, long lda,
                                          long ldc, int splits, int form, const float* row_sumsq, int row_parts,
                                          float row_count, float row_eps, float* residual, const float* norm_weight,
-                                         float* sumsq_out, int* error_flag, cudaStream_t stream) {
+                                         float* sumsq_out, float gate_limit, float gate_slope, int* error_flag, cudaStream_t stream) {
     Epilogue ep{row_sumsq, row_sumsq ? row_parts : 0, row_count, row_eps, nullptr, nullptr, nullptr, g_gemm_stamps};
     if (g_gemm_stamps) g_gemm_stamps += 8 * 1024;  // the next launch's stamps follow (up to 1,024 CTAs a launch)
     if (row_sumsq && row_parts <= 0) return KIRAI_ERR_BAD_SIZE;
@@ -1302,6 +1303,10 @@ KIRAI_EXPORT int kirai_gemm_bf16_general(const void* A, const void* W, int tiled
         case 2: return gemm_dispatch<bf16, 1>(A, W, tiled != 0, C, M, N, K, lda, ldc, splits, ep, error_flag, stream);
         case 5:
             ep.gate_act = 1;
+            return gemm_dispatch<bf16, 1>(A, W, tiled != 0, C, M, N, K, lda, ldc, splits, ep, error_flag, stream);
+        case 7:
+            if (!(gate_limit > 0.0f)) return KIRAI_ERR_BAD_SIZE;
+            ep.gate_act = 2, ep.gate_limit = gate_limit, ep.gate_slope = gate_slope;
             return gemm_dispatch<bf16, 1>(A, W, tiled != 0, C, M, N, K, lda, ldc, splits, ep, error_flag, stream);
         case 4: return gemm_dispatch<bf16, 3>(A, W, tiled != 0, C, M, N, K, lda, ldc, splits, ep, error_flag, stream);
         case 3:

@@ -1,7 +1,7 @@
 // Row-wise kernels of layer forms beside the pre-norm / rotary ones of elementwise.cu:
 //
 //   * embedding rows times a constant, plus a sinusoidal position vector (column 2i the sine and column 2i + 1
-//     the cosine of position * frequency[i], angles in 32-bit);
+//     the cosine of position * frequency[i], angles in 32-bit), or plus a learned vector per position;
 //   * the norm on a sub-layer's OUTPUT: stream += y / sqrt(mean(y^2) + eps) * w, with the runtime-dtype copy of the
 //     new stream that the next sub-layer reads written in the same pass; the same followed by the norm that reads the
 //     stream next (norm_add_norm), and with the stream's copy written into a run of columns of a wider buffer
@@ -19,8 +19,8 @@
 template <typename T, typename C>
 __global__ void embedding_sinusoid_kernel(const T* __restrict__ table, const int* __restrict__ ids,
                                           const int* __restrict__ positions, const float* __restrict__ freq,
-                                          float* __restrict__ out, C* __restrict__ copy, int hidden, int vocab,
-                                          float scale, int* __restrict__ error_flag) {
+                                          const T* __restrict__ pos_table, int pos_rows, float* __restrict__ out,
+                                          C* __restrict__ copy, int hidden, int vocab, float scale, int* __restrict__ error_flag) {
     pdl_launch_dependents();
     pdl_wait();
     const int token = blockIdx.x;
@@ -31,6 +31,15 @@ __global__ void embedding_sinusoid_kernel(const T* __restrict__ table, const int
     }
     const float pos = freq ? (float)positions[token] : 0.0f;
     const T* row = table + (size_t)id * hidden;
+    const T* pos_row = nullptr;
+    if (pos_table) {
+        const int position = positions[token];
+        if (position < 0 || position >= pos_rows) {
+            if (threadIdx.x == 0) atomicExch(error_flag, KIRAI_FLAG_BAD_POSITION);
+            return;
+        }
+        pos_row = pos_table + (size_t)position * hidden;
+    }
     float* dst = out + (size_t)token * hidden;
     C* dst_copy = copy ? copy + (size_t)token * hidden : nullptr;
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
@@ -39,6 +48,7 @@ __global__ void embedding_sinusoid_kernel(const T* __restrict__ table, const int
             const float angle = pos * freq[i >> 1];
             v += (i & 1) ? cosf(angle) : sinf(angle);
         }
+        if (pos_row) v += to_f32<T>(pos_row[i]);
         dst[i] = v;
         if (dst_copy) dst_copy[i] = from_f32<C>(v);
     }
@@ -46,24 +56,25 @@ __global__ void embedding_sinusoid_kernel(const T* __restrict__ table, const int
 
 template <typename T>
 static int embedding_sinusoid_launch(const void* table, const int* ids, const int* positions, const float* freq,
-                                     float* out, void* copy, int tokens, int hidden, int vocab, float scale,
+                                     const void* pos_table, int pos_rows, float* out, void* copy, int tokens, int hidden, int vocab, float scale,
                                      int* error_flag, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     return launch_pdl(embedding_sinusoid_kernel<T, bf16>, dim3(tokens), dim3(256), 0, stream, 1u, (const T*)table, ids,
-                      positions, freq, out, (bf16*)copy, hidden, vocab, scale, error_flag);
+                      positions, freq, (const T*)pos_table, pos_rows, out, (bf16*)copy, hidden, vocab, scale, error_flag);
 }
 
-// out [T, H] (float32) = table[id] * scale (+ the sinusoid of the token's position when freq [ceil(H/2)] is given);
+// out [T, H] (float32) = table[id] * scale (+ the sinusoid of the token's position when freq [ceil(H/2)] is given, + row
+// `position` of pos_table [pos_rows, H] when that is given);
 // copy (bf16, may be null) receives the same rows rounded.
 KIRAI_EXPORT int kirai_embedding_sinusoid_f32(const void* table, const int* ids, const int* positions, const float* freq,
-                                              float* out, void* copy, int tokens, int hidden, int vocab, float scale,
+                                              const void* pos_table, int pos_rows, float* out, void* copy, int tokens, int hidden, int vocab, float scale,
                                               int* error_flag, cudaStream_t stream) {
-    return embedding_sinusoid_launch<float>(table, ids, positions, freq, out, copy, tokens, hidden, vocab, scale, error_flag, stream);
+    return embedding_sinusoid_launch<float>(table, ids, positions, freq, pos_table, pos_rows, out, copy, tokens, hidden, vocab, scale, error_flag, stream);
 }
 KIRAI_EXPORT int kirai_embedding_sinusoid_bf16(const void* table, const int* ids, const int* positions, const float* freq,
-                                               float* out, void* copy, int tokens, int hidden, int vocab, float scale,
+                                               const void* pos_table, int pos_rows, float* out, void* copy, int tokens, int hidden, int vocab, float scale,
                                                int* error_flag, cudaStream_t stream) {
-    return embedding_sinusoid_launch<bf16>(table, ids, positions, freq, out, copy, tokens, hidden, vocab, scale, error_flag, stream);
+    return embedding_sinusoid_launch<bf16>(table, ids, positions, freq, pos_table, pos_rows, out, copy, tokens, hidden, vocab, scale, error_flag, stream);
 }
 
 // ------------------------------------------------------- norm on the output

@@ -8,8 +8,9 @@
 //     as a walk over a request's tokens (steps of few tokens) and as a scan over pieces of SCAN_PIECE tokens
 //     (prompt portions): the pieces' (product of 1 - z, end state from zero) first, then every piece's incoming
 //     state, then the rows;
-//   * the preparation of attention with biases, a rotation of a part of each head and a factor per head: queries
-//     out (heads padded to the cache's row width), keys and values to their pages;
+//   * the preparation of attention with biases, a norm per head, a rotation of a part of each head and a factor per head:
+//     queries out (heads padded to the cache's row width), keys and values to their pages;
+//   * the difference of two attention maps over the same values, normed per head;
 //   * the preparation of latent attention: RMS norms of the query latent and of the key/value latent, rotation of
 //     the shared key part, the latent row to the pages (as key row [latent, rotated part] and as value row [latent]);
 //   * small element-wise steps: a sigmoid gate on padded heads, a gated activation, a bias on rows.
@@ -484,23 +485,64 @@ KIRAI_EXPORT int kirai_mingru_bf16(const float* zxg, long row_stride, const floa
                                max_query_len, width, num_slots, walk_limit, stream);
 }
 
-// ------------------------------------- attention preparation: bias, rotation, factor
+// --------------------------- attention preparation: bias, per-head norm, rotation, factor
 // One block per token.  qkv row (float32): nq heads of dk, then nkv heads of dk, then nkv heads of dv (further
-// columns, as an output gate's, are not touched).  Columns [rot_off, rot_off + rot_dims) of every query and key head
-// are rotated, column i of the first half with column i + rot_dims / 2, by position * inv_freq[i]; query head h is
-// multiplied by q_factor[h]; cosine and sine are multiplied by rot_amp (1: a plain rotation).  Queries leave as [nq, dpad] rows with zeros beyond dk; keys and values go to the
-// token's row of its page, cache [pages, 2, nkv, page, dpad].
+// columns, as an output gate's, are not touched).  With q_norm / k_norm [dk] every query / key head is divided by its root
+// mean square (eps inside the root) and multiplied by that weight, which the heads share.  Columns [rot_off, rot_off +
+// rot_dims) of every query and key head are rotated, column i of the first half with column i + rot_dims / 2, by position *
+// inv_freq[i]; query head h is multiplied by q_factor[h]; cosine and sine are multiplied by rot_amp (1: a plain rotation).
+// Queries leave as [nq, dpad] rows with zeros beyond dk; keys and values go to the token's row of its page, cache
+// [pages, 2, nkv, page, dpad].  keys_as_values: there are no value columns, the value row is the key head as projected
+// (with its bias), ahead of norm and rotation.  q_maps m > 1: a head's dk columns are m queries of dk / m columns side by
+// side (as its key row is m keys side by side); every one leaves as a row of its own, [nq, m, dpad], in its own columns
+// and zero elsewhere, so that its product with the key row is its product with its own key.
+struct HeadsPrepare {
+    const float* qkv;
+    long qkv_stride;
+    const float *q_bias, *k_bias, *v_bias, *q_factor, *q_norm, *k_norm, *inv_freq;
+    float eps;
+    int rot_off, rot_dims;
+    float rot_amp;
+    const int *block_table, *request_of_token, *positions;
+    int q_heads, kv_heads, dk, dv, dpad, q_maps, keys_as_values;
+    int page_size, table_width, num_pages;
+    int* error_flag;
+};
+
+// Where a token's rows of the cache start (kv head 0's key row), or -1.
+__device__ __forceinline__ long prepared_page_base(const HeadsPrepare& p, int token, int position) {
+    if (p.kv_heads <= 0) return -1;
+    const int logical = position / p.page_size;
+    const int page = logical < p.table_width ? p.block_table[(long)p.request_of_token[token] * p.table_width + logical] : -1;
+    if (page < 0 || page >= p.num_pages) {
+        if (threadIdx.x == 0) atomicExch(p.error_flag, KIRAI_FLAG_NO_PAGE_WRITE);
+        return -1;
+    }
+    return (((long)page * 2) * p.kv_heads * p.page_size + (position % p.page_size)) * (long)p.dpad;
+}
+
 template <typename T>
 __device__ __forceinline__ void rotate_head_to(const float* __restrict__ src, const float* __restrict__ bias, T* __restrict__ dst,
                                                int width, int rot_off, int rot_dims, const float* __restrict__ inv_freq,
-                                               float pos, float factor, int lane, int lanes, float rot_amp = 1.0f) {
+                                               float pos, float factor, int lane, int lanes, float rot_amp,
+                                               const float* __restrict__ norm, float eps) {
     const int half = rot_dims >> 1;
+    if (norm) {
+        float acc = 0.0f;
+        for (int c = lane; c < width; c += lanes) {
+            const float v = src[c] + (bias ? bias[c] : 0.0f);
+            acc = fmaf(v, v, acc);
+        }
+        const float variance = warp_sum(acc) / (float)width + eps;
+        factor *= variance == 0.0f ? 0.0f : 1.0f / sqrtf(variance);
+    }
     for (int c = lane; c < width; c += lanes) {
         const int r = c - rot_off;
         if (r >= 0 && r < rot_dims) {
             if (r >= half) continue;  // written with its partner
-            const float u = src[c] + (bias ? bias[c] : 0.0f);
-            const float v = src[c + half] + (bias ? bias[c + half] : 0.0f);
+            float u = src[c] + (bias ? bias[c] : 0.0f);
+            float v = src[c + half] + (bias ? bias[c + half] : 0.0f);
+            if (norm) u *= norm[c], v *= norm[c + half];
             float sn, cs;
             sincosf(pos * inv_freq[r], &sn, &cs);
             sn *= rot_amp;
@@ -508,93 +550,255 @@ __device__ __forceinline__ void rotate_head_to(const float* __restrict__ src, co
             dst[c] = from_f32<T>((u * cs - v * sn) * factor);
             dst[c + half] = from_f32<T>((v * cs + u * sn) * factor);
         } else {
-            dst[c] = from_f32<T>((src[c] + (bias ? bias[c] : 0.0f)) * factor);
+            const float v = src[c] + (bias ? bias[c] : 0.0f);
+            dst[c] = from_f32<T>((norm ? v * norm[c] : v) * factor);
         }
     }
 }
 
 template <typename T>
-__global__ void qkv_rope_write_kernel(const float* __restrict__ qkv, long qkv_stride, const float* __restrict__ q_bias,
-                                      const float* __restrict__ k_bias, const float* __restrict__ v_bias,
-                                      const float* __restrict__ q_factor, const float* __restrict__ inv_freq, int rot_off,
-                                      int rot_dims, float rot_amp, T* __restrict__ q_out, T* __restrict__ cache,
-                                      const int* __restrict__ block_table, const int* __restrict__ request_of_token,
-                                      const int* __restrict__ positions, int q_heads, int kv_heads, int dk, int dv, int dpad,
-                                      int page_size, int table_width, int num_pages, int* __restrict__ error_flag) {
+__global__ void qkv_rope_write_kernel(HeadsPrepare p, T* __restrict__ q_out, T* __restrict__ cache) {
     pdl_launch_dependents();
     const int token = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-    const int position = positions[token];
-    long page_base = -1;
-    if (kv_heads > 0) {
-        const int logical = position / page_size;
-        const int page = logical < table_width ? block_table[(long)request_of_token[token] * table_width + logical] : -1;
-        if (page < 0 || page >= num_pages) {
-            if (threadIdx.x == 0) atomicExch(error_flag, KIRAI_FLAG_NO_PAGE_WRITE);
-        } else {
-            page_base = (((long)page * 2) * kv_heads * page_size + (position % page_size)) * (long)dpad;
-        }
-    }
+    const int position = p.positions[token];
+    const long page_base = prepared_page_base(p, token, position);
     pdl_wait();
     const float pos = (float)position;
-    const float* src = qkv + (size_t)token * qkv_stride;
-    const long head_rows = (long)page_size * dpad;
+    const float* src = p.qkv + (size_t)token * p.qkv_stride;
+    const int dk = p.dk, dv = p.dv, dpad = p.dpad, maps = p.q_maps, part = dk / maps;
+    const long head_rows = (long)p.page_size * dpad;
     // a warp per head: query heads, then key heads, then value heads
-    for (int unit = warp; unit < q_heads + 2 * kv_heads; unit += warps) {
-        if (unit < q_heads) {
-            T* dst = q_out + ((size_t)token * q_heads + unit) * dpad;
-            rotate_head_to<T>(src + (size_t)unit * dk, q_bias ? q_bias + (size_t)unit * dk : nullptr, dst, dk, rot_off, rot_dims,
-                              inv_freq, pos, q_factor ? q_factor[unit] : 1.0f, lane, 32, rot_amp);
-            for (int c = dk + lane; c < dpad; c += 32) dst[c] = from_f32<T>(0.0f);
-        } else if (page_base >= 0 && unit < q_heads + kv_heads) {
-            const int head = unit - q_heads;
-            rotate_head_to<T>(src + (size_t)q_heads * dk + (size_t)head * dk, k_bias ? k_bias + (size_t)head * dk : nullptr,
-                              cache + page_base + head * head_rows, dk, rot_off, rot_dims, inv_freq, pos, 1.0f, lane, 32, rot_amp);
+    for (int unit = warp; unit < p.q_heads + 2 * p.kv_heads; unit += warps) {
+        if (unit < p.q_heads) {
+            const float* q = src + (size_t)unit * dk;
+            const float* bias = p.q_bias ? p.q_bias + (size_t)unit * dk : nullptr;
+            const float factor = p.q_factor ? p.q_factor[unit] : 1.0f;
+            T* dst = q_out + ((size_t)token * p.q_heads + unit) * maps * dpad;
+            if (maps == 1) {
+                rotate_head_to<T>(q, bias, dst, dk, p.rot_off, p.rot_dims, p.inv_freq, pos, factor, lane, 32, p.rot_amp, p.q_norm, p.eps);
+                for (int c = dk + lane; c < dpad; c += 32) dst[c] = from_f32<T>(0.0f);
+            } else {
+                for (int at = lane; at < maps * dpad; at += 32) {
+                    const int m = at / dpad, c = at - m * dpad;
+                    const bool own = c >= m * part && c < (m + 1) * part;
+                    dst[at] = from_f32<T>(own ? (q[c] + (bias ? bias[c] : 0.0f)) * factor : 0.0f);
+                }
+            }
+        } else if (page_base >= 0 && unit < p.q_heads + p.kv_heads) {
+            const int head = unit - p.q_heads;
+            rotate_head_to<T>(src + (size_t)p.q_heads * dk + (size_t)head * dk, p.k_bias ? p.k_bias + (size_t)head * dk : nullptr,
+                              cache + page_base + head * head_rows, dk, p.rot_off, p.rot_dims, p.inv_freq, pos, 1.0f, lane, 32, p.rot_amp,
+                              p.k_norm, p.eps);
         } else if (page_base >= 0) {
-            const int head = unit - q_heads - kv_heads;
-            const float* v = src + (size_t)(q_heads + kv_heads) * dk + (size_t)head * dv;
-            T* dst = cache + page_base + (long)kv_heads * head_rows + head * head_rows;
-            for (int c = lane; c < dv; c += 32) dst[c] = from_f32<T>(v[c] + (v_bias ? v_bias[(size_t)head * dv + c] : 0.0f));
+            const int head = unit - p.q_heads - p.kv_heads;
+            const float* v = src + (size_t)(p.q_heads + (p.keys_as_values ? 0 : p.kv_heads)) * dk + (size_t)head * dv;
+            const float* bias = p.keys_as_values ? p.k_bias : p.v_bias;
+            T* dst = cache + page_base + (long)p.kv_heads * head_rows + head * head_rows;
+            for (int c = lane; c < dv; c += 32) dst[c] = from_f32<T>(v[c] + (bias ? bias[(size_t)head * dv + c] : 0.0f));
+        }
+    }
+}
+
+// The same without a rotation, four columns at a time (every width, stride and pointer allows 16-byte accesses); a warp
+// per head keeps up to 512 columns in registers between the statistics and the stores.  A key head whose values are the
+// keys is read once for both rows.
+template <typename T>
+__global__ void heads_write_vec_kernel(HeadsPrepare p, T* __restrict__ q_out, T* __restrict__ cache) {
+    pdl_launch_dependents();
+    const int token = blockIdx.x;
+    const int lane = threadIdx.x & 31, warp = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5), warps = gridDim.y * (blockDim.x >> 5);
+    const int position = p.positions[token];
+    const long page_base = prepared_page_base(p, token, position);
+    pdl_wait();
+    const float* src = p.qkv + (size_t)token * p.qkv_stride;
+    const int dk = p.dk, dv = p.dv, dpad = p.dpad, maps = p.q_maps, part = dk / maps;
+    const long head_rows = (long)p.page_size * dpad;
+    const int units = p.q_heads + (p.keys_as_values ? 1 : 2) * p.kv_heads;
+    for (int unit = warp; unit < units; unit += warps) {
+        const bool query = unit < p.q_heads, value = unit >= p.q_heads + p.kv_heads;
+        if (!query && page_base < 0) continue;
+        const int head = query ? unit : (value ? unit - p.q_heads - p.kv_heads : unit - p.q_heads);
+        const int width = value ? dv : dk;
+        const float* row = src + (query ? (size_t)head * dk : value ? (size_t)(p.q_heads + p.kv_heads) * dk + (size_t)head * dv
+                                                                    : (size_t)(p.q_heads + head) * dk);
+        const float* bias = query ? p.q_bias : (value ? p.v_bias : p.k_bias);
+        const float* norm = query ? p.q_norm : (value ? nullptr : p.k_norm);
+        float kept[4][4];
+        float acc = 0.0f;
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+            const int c = (lane + 32 * n) * 4;
+            if (c >= width) break;
+            load4<float>(row + c, kept[n]);
+            if (bias) {
+                float add[4];
+                load4<float>(bias + (size_t)head * width + c, add);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) kept[n][j] += add[j];
+            }
+            acc += (kept[n][0] * kept[n][0] + kept[n][1] * kept[n][1]) + (kept[n][2] * kept[n][2] + kept[n][3] * kept[n][3]);
+        }
+        T* dst = query ? q_out + ((size_t)token * p.q_heads + head) * maps * dpad
+                       : cache + page_base + ((value ? (long)p.kv_heads : 0L) + head) * head_rows;
+        if (!query && !value && p.keys_as_values) {
+            T* v_dst = dst + (long)p.kv_heads * head_rows;
+#pragma unroll
+            for (int n = 0; n < 4; ++n) {
+                const int c = (lane + 32 * n) * 4;
+                if (c < width) store4<T>(v_dst + c, kept[n]);
+            }
+        }
+        float factor = query && p.q_factor ? p.q_factor[head] : 1.0f;
+        if (norm) {
+            const float variance = warp_sum(acc) / (float)width + p.eps;
+            factor *= variance == 0.0f ? 0.0f : 1.0f / sqrtf(variance);
+        }
+        const float zero[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+            const int c = (lane + 32 * n) * 4;
+            if (c < width) {
+                float w[4] = {1.0f, 1.0f, 1.0f, 1.0f};
+                if (norm) load4<float>(norm + c, w);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) kept[n][j] *= factor * w[j];
+                if (!query || maps == 1) {
+                    store4<T>(dst + c, kept[n]);
+                } else {
+                    const int own = c / part;
+                    for (int m = 0; m < maps; ++m) {
+                        if (m == own) store4<T>(dst + m * dpad + c, kept[n]);
+                        else store4<T>(dst + m * dpad + c, zero);
+                    }
+                }
+            } else if (query && c < dpad) {
+                for (int m = 0; m < maps; ++m) store4<T>(dst + m * dpad + c, zero);
+            }
         }
     }
 }
 
 template <typename T>
-static int qkv_rope_write_launch(const float* qkv, long qkv_stride, const float* q_bias, const float* k_bias, const float* v_bias,
-                                 const float* q_factor, const float* inv_freq, int rot_off, int rot_dims, float rot_amp, void* q_out, void* cache,
-                                 const int* block_table, const int* request_of_token, const int* positions, int tokens,
-                                 int q_heads, int kv_heads, int dk, int dv, int dpad, int page_size, int table_width,
-                                 int num_pages, int* error_flag, cudaStream_t stream) {
+static int qkv_rope_write_launch(const HeadsPrepare& p, void* q_out, void* cache, int tokens, cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (q_heads <= 0 || kv_heads < 0 || dk <= 0 || dv <= 0 || dpad < dk || dpad < dv || page_size <= 0) return KIRAI_ERR_BAD_SIZE;
-    if (rot_dims < 0 || rot_dims % 2 || rot_off < 0 || rot_off + rot_dims > dk || (rot_dims > 0 && !inv_freq)) return KIRAI_ERR_BAD_SIZE;
-    if (kv_heads > 0 && !cache) return KIRAI_ERR_BAD_SIZE;
-    const int units = q_heads + 2 * kv_heads;
+    if (p.q_heads <= 0 || p.kv_heads < 0 || p.dk <= 0 || p.dv <= 0 || p.dpad < p.dk || p.dpad < p.dv || p.page_size <= 0) return KIRAI_ERR_BAD_SIZE;
+    if (p.rot_dims < 0 || p.rot_dims % 2 || p.rot_off < 0 || p.rot_off + p.rot_dims > p.dk || (p.rot_dims > 0 && !p.inv_freq)) return KIRAI_ERR_BAD_SIZE;
+    if (p.kv_heads > 0 && !cache) return KIRAI_ERR_BAD_SIZE;
+    if (p.q_maps < 1 || p.dk % p.q_maps) return KIRAI_ERR_BAD_SIZE;
+    if (p.q_maps > 1 && (p.q_norm || p.rot_dims)) return KIRAI_ERR_UNSUPPORTED;  // a norm or a rotation over one map's columns
+    if (p.keys_as_values && p.dv != p.dk) return KIRAI_ERR_BAD_SIZE;
+    const bool vec = p.rot_dims == 0 && p.dk % 4 == 0 && p.dv % 4 == 0 && p.dpad % 4 == 0 && p.dpad <= 512 && (p.dk / p.q_maps) % 4 == 0 &&
+                     p.qkv_stride % 4 == 0 &&
+                     (((uintptr_t)p.qkv | (uintptr_t)p.q_bias | (uintptr_t)p.k_bias | (uintptr_t)p.v_bias | (uintptr_t)p.q_norm |
+                       (uintptr_t)p.k_norm | (uintptr_t)q_out | (uintptr_t)cache) & 15) == 0;
+    const int units = p.q_heads + 2 * p.kv_heads;
     const int threads = units >= 8 ? 256 : 32 * units;
-    return launch_pdl(qkv_rope_write_kernel<T>, dim3(tokens), dim3(threads), 0, stream, 1u, qkv, qkv_stride, q_bias, k_bias, v_bias,
-                      q_factor, inv_freq, rot_off, rot_dims, rot_amp, (T*)q_out, (T*)cache, block_table, request_of_token, positions,
-                      q_heads, kv_heads, dk, dv, dpad, page_size, table_width, num_pages, error_flag);
+    if (vec) {
+        // few tokens: a token's heads spread over more blocks
+        const unsigned spread = tokens >= 256 ? 1u : (unsigned)((units + 7) / 8);
+        return launch_pdl(heads_write_vec_kernel<T>, dim3(tokens, spread), dim3(threads), 0, stream, 1u, p, (T*)q_out, (T*)cache);
+    }
+    return launch_pdl(qkv_rope_write_kernel<T>, dim3(tokens), dim3(threads), 0, stream, 1u, p, (T*)q_out, (T*)cache);
 }
 
-KIRAI_EXPORT int kirai_qkv_rope_write_f32(const float* qkv, long qkv_stride, const float* q_bias, const float* k_bias,
-                                          const float* v_bias, const float* q_factor, const float* inv_freq, int rot_off,
-                                          int rot_dims, float rot_amp, void* q_out, void* cache, const int* block_table,
-                                          const int* request_of_token, const int* positions, int tokens, int q_heads,
-                                          int kv_heads, int dk, int dv, int dpad, int page_size, int table_width,
-                                          int num_pages, int* error_flag, cudaStream_t stream) {
-    return qkv_rope_write_launch<float>(qkv, qkv_stride, q_bias, k_bias, v_bias, q_factor, inv_freq, rot_off, rot_dims, rot_amp, q_out,
-                                        cache, block_table, request_of_token, positions, tokens, q_heads, kv_heads, dk, dv, dpad,
-                                        page_size, table_width, num_pages, error_flag, stream);
+#define KIRAI_QKV_ROPE_WRITE(NAME, T)                                                                                             \
+    KIRAI_EXPORT int NAME(const float* qkv, long qkv_stride, const float* q_bias, const float* k_bias, const float* v_bias,       \
+                          const float* q_factor, const float* q_norm, const float* k_norm, float eps, const float* inv_freq,      \
+                          int rot_off, int rot_dims, float rot_amp, void* q_out, void* cache, const int* block_table,            \
+                          const int* request_of_token, const int* positions, int tokens, int q_heads, int kv_heads, int dk,      \
+                          int dv, int dpad, int q_maps, int keys_as_values, int page_size, int table_width, int num_pages,       \
+                          int* error_flag, cudaStream_t stream) {                                                                \
+        const HeadsPrepare p{qkv, qkv_stride, q_bias, k_bias, v_bias, q_factor, q_norm, k_norm, inv_freq, eps, rot_off, rot_dims, \
+                             rot_amp, block_table, request_of_token, positions, q_heads, kv_heads, dk, dv, dpad, q_maps,         \
+                             keys_as_values, page_size, table_width, num_pages, error_flag};                                     \
+        return qkv_rope_write_launch<T>(p, q_out, cache, tokens, stream);                                                        \
+    }
+KIRAI_QKV_ROPE_WRITE(kirai_qkv_rope_write_f32, float)
+KIRAI_QKV_ROPE_WRITE(kirai_qkv_rope_write_bf16, bf16)
+#undef KIRAI_QKV_ROPE_WRITE
+
+// ---------------------------------------------------- two attention maps made one
+// A warp per (token, head).  x [T, heads, 2, dpad]: the outputs of a head's two attention maps over the same values, the
+// first `used` columns of a row count.  o = first - lambda * second, divided by its root mean square over the head's
+// columns (eps inside the root), times `factor`; out [T, heads * used].
+template <typename T>
+__global__ void map_difference_kernel(const T* __restrict__ x, T* __restrict__ out, long units, int used, int dpad, float lambda, float eps,
+                                      float factor) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const long unit = blockIdx.x * (long)(blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (unit >= units) return;
+    const T* a = x + unit * 2 * dpad;
+    const T* b = a + dpad;
+    T* o = out + unit * used;
+    float acc = 0.0f;
+    for (int c = lane; c < used; c += 32) {
+        const float v = fmaf(-lambda, to_f32<T>(b[c]), to_f32<T>(a[c]));
+        acc = fmaf(v, v, acc);
+    }
+    const float variance = warp_sum(acc) / (float)used + eps;
+    const float scale = variance == 0.0f ? 0.0f : factor / sqrtf(variance);
+    for (int c = lane; c < used; c += 32) o[c] = from_f32<T>(fmaf(-lambda, to_f32<T>(b[c]), to_f32<T>(a[c])) * scale);
 }
-KIRAI_EXPORT int kirai_qkv_rope_write_bf16(const float* qkv, long qkv_stride, const float* q_bias, const float* k_bias,
-                                           const float* v_bias, const float* q_factor, const float* inv_freq, int rot_off,
-                                           int rot_dims, float rot_amp, void* q_out, void* cache, const int* block_table,
-                                           const int* request_of_token, const int* positions, int tokens, int q_heads,
-                                           int kv_heads, int dk, int dv, int dpad, int page_size, int table_width,
-                                           int num_pages, int* error_flag, cudaStream_t stream) {
-    return qkv_rope_write_launch<bf16>(qkv, qkv_stride, q_bias, k_bias, v_bias, q_factor, inv_freq, rot_off, rot_dims, rot_amp, q_out,
-                                       cache, block_table, request_of_token, positions, tokens, q_heads, kv_heads, dk, dv, dpad,
-                                       page_size, table_width, num_pages, error_flag, stream);
+
+// The same four columns at a time, up to 512 columns, the head in registers between the statistics and the output.
+template <typename T>
+__global__ void map_difference_vec_kernel(const T* __restrict__ x, T* __restrict__ out, long units, int used, int dpad, float lambda,
+                                          float eps, float factor) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const long unit = blockIdx.x * (long)(blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (unit >= units) return;
+    const T* a = x + unit * 2 * dpad;
+    float kept[4][4];
+    float acc = 0.0f;
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+        const int c = (lane + 32 * n) * 4;
+        if (c >= used) break;
+        float b[4];
+        load4<T>(a + c, kept[n]);
+        load4<T>(a + dpad + c, b);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            kept[n][j] = fmaf(-lambda, b[j], kept[n][j]);
+            acc = fmaf(kept[n][j], kept[n][j], acc);
+        }
+    }
+    const float variance = warp_sum(acc) / (float)used + eps;
+    const float scale = variance == 0.0f ? 0.0f : factor / sqrtf(variance);
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+        const int c = (lane + 32 * n) * 4;
+        if (c >= used) break;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) kept[n][j] *= scale;
+        store4<T>(out + unit * used + c, kept[n]);
+    }
+}
+
+template <typename T>
+static int map_difference_launch(const void* x, void* out, int rows, int heads, int used, int dpad, float lambda, float eps, float factor,
+                                 cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (heads <= 0 || used <= 0 || dpad < used) return KIRAI_ERR_BAD_SIZE;
+    const long units = (long)rows * heads;
+    const unsigned blocks = (unsigned)((units + 7) / 8);
+    const bool vec = used % 4 == 0 && dpad % 4 == 0 && used <= 512 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0;
+    return launch_pdl(vec ? map_difference_vec_kernel<T> : map_difference_kernel<T>, dim3(blocks), dim3(256), 0, stream, 1u, (const T*)x,
+                      (T*)out, units, used, dpad, lambda, eps, factor);
+}
+
+KIRAI_EXPORT int kirai_map_difference_f32(const void* x, void* out, int rows, int heads, int used, int dpad, float lambda, float eps,
+                                          float factor, cudaStream_t stream) {
+    return map_difference_launch<float>(x, out, rows, heads, used, dpad, lambda, eps, factor, stream);
+}
+KIRAI_EXPORT int kirai_map_difference_bf16(const void* x, void* out, int rows, int heads, int used, int dpad, float lambda, float eps,
+                                           float factor, cudaStream_t stream) {
+    return map_difference_launch<bf16>(x, out, rows, heads, used, dpad, lambda, eps, factor, stream);
 }
 
 // --------------------------------------------------- latent attention preparation

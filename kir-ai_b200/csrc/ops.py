@@ -28,6 +28,7 @@ _ERROR_NAMES = {
     3: "a key position has no page in its request's block table (attention read)",
     4: "a bounded wait inside a kernel ran out",
     5: "a row of logits has no maximum (every entry is NaN or -inf); token 0 was written for it",
+    6: "a token's position is beyond the table of learned positions",
 }
 
 _REFUSALS = {
@@ -276,10 +277,12 @@ def rope_(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor, rota
 
 # ------------------------------------------------- forms of other layer designs
 def embedding_scaled(table: torch.Tensor, ids: torch.Tensor, scale: float, positions: Optional[torch.Tensor] = None,
-                     frequencies: Optional[torch.Tensor] = None, copy_dtype: Optional[torch.dtype] = None):
+                     frequencies: Optional[torch.Tensor] = None, copy_dtype: Optional[torch.dtype] = None,
+                     position_table: Optional[torch.Tensor] = None):
     """Rows ``ids`` of the row-major ``table`` [V, H] times ``scale`` as the 32-bit stream [T, H]; with ``frequencies``
     [ceil(H / 2)] (float32) the sinusoid of each token's position is added: column 2i gets sin(position * f_i), column
-    2i + 1 the cosine.  Returns (stream, copy): ``copy`` is the stream rounded to bfloat16 when ``copy_dtype`` asks for
+    2i + 1 the cosine; with ``position_table`` [P, H] (the dtype of ``table``) its row of the token's position is added
+    (unscaled; a position beyond the table sets the error word).  Returns (stream, copy): ``copy`` is the stream rounded to bfloat16 when ``copy_dtype`` asks for
     it, else None."""
     _need_cuda(table, ids, positions, frequencies)
     assert ids.dtype == torch.int32 and ids.is_contiguous() and table.dim() == 2 and table.is_contiguous()
@@ -287,12 +290,16 @@ def embedding_scaled(table: torch.Tensor, ids: torch.Tensor, scale: float, posit
     if frequencies is not None:
         assert positions is not None and positions.dtype == torch.int32 and positions.numel() == tokens and positions.is_contiguous()
         assert frequencies.dtype == torch.float32 and frequencies.numel() == (hidden + 1) // 2 and frequencies.is_contiguous()
+    if position_table is not None:
+        _need_cuda(position_table)
+        assert positions is not None and positions.dtype == torch.int32 and positions.numel() == tokens and positions.is_contiguous()
+        assert position_table.dtype == table.dtype and position_table.dim() == 2 and position_table.shape[1] == hidden and position_table.is_contiguous()
     out = torch.empty((tokens, hidden), dtype=torch.float32, device=table.device)
     copy = None
     if copy_dtype == torch.bfloat16:
         copy = torch.empty((tokens, hidden), dtype=torch.bfloat16, device=table.device)
     _call(f"kirai_embedding_sinusoid_{_suffix(table.dtype)}", _ptr(table), _ptr(ids), _ptr(positions), _ptr(frequencies),
-          _ptr(out), _ptr(copy), _i(tokens), _i(hidden), _i(table.shape[0]), _f(scale), _ptr(error_flag(table.device)), _stream())
+          _ptr(position_table), _i(position_table.shape[0] if position_table is not None else 0), _ptr(out), _ptr(copy), _i(tokens), _i(hidden), _i(table.shape[0]), _f(scale), _ptr(error_flag(table.device)), _stream())
     return out, copy
 
 
@@ -381,17 +388,23 @@ def head_linear_gate(x: torch.Tensor, weight: torch.Tensor, heads: int, used: in
     return out
 
 
+def _block_tiles(device: torch.device, groups: int, padded: int) -> torch.Tensor:
+    """The group of every 128-row tile of rows laid out group by group, ``padded`` rows (a multiple of 128) each."""
+    key = (device, groups, padded)
+    tile_group = _head_tiles.get(key)
+    if tile_group is None:  # tile i belongs to group i // (padded / 128)
+        if len(_head_tiles) > 64:
+            _head_tiles.clear()
+        tile_group = (torch.arange(groups * (padded // 128), dtype=torch.int32) // (padded // 128)).to(torch.int32).to(device)
+        _head_tiles[key] = tile_group
+    return tile_group
+
+
 def _head_linear_gate_grouped(x: torch.Tensor, padded_weight: torch.Tensor, heads: int, n: int, gate: Optional[torch.Tensor]) -> torch.Tensor:
     tokens, pad = x.shape[0], x.shape[1] // heads
     padded = -(-tokens // 128) * 128
     assert padded_weight.dtype == torch.bfloat16 and padded_weight.shape == (heads * n, pad) and padded_weight.is_contiguous()
-    key = (x.device, heads, padded)
-    tile_group = _head_tiles.get(key)
-    if tile_group is None:  # tile i of the head-major rows belongs to head i // (padded / 128)
-        if len(_head_tiles) > 64:
-            _head_tiles.clear()
-        tile_group = (torch.arange(heads * (padded // 128), dtype=torch.int32) // (padded // 128)).to(torch.int32).to(x.device)
-        _head_tiles[key] = tile_group
+    tile_group = _block_tiles(x.device, heads, padded)
     rows = torch.empty((heads * padded, pad), dtype=torch.bfloat16, device=x.device)
     _call("kirai_head_major_bf16", _ptr(x), _ptr(rows), _i(tokens), _i(padded), _i(heads), _i(pad), _stream())
     y = linear_grouped(rows, padded_weight, heads, tile_group, out_dtype=torch.float32)
@@ -523,17 +536,23 @@ def qkv_rope_write(qkv: torch.Tensor, q_heads: int, kv_heads: int, key_dim: int,
                    q_bias: Optional[torch.Tensor], k_bias: Optional[torch.Tensor], v_bias: Optional[torch.Tensor],
                    q_factor: Optional[torch.Tensor], inv_freq: Optional[torch.Tensor], rot_offset: int, rot_dims: int,
                    cache: Optional[torch.Tensor], block_table: torch.Tensor, request_of_token: torch.Tensor,
-                   positions: torch.Tensor, out_dtype: torch.dtype, rot_amplitude: float = 1.0) -> torch.Tensor:
+                   positions: torch.Tensor, out_dtype: torch.dtype, rot_amplitude: float = 1.0,
+                   q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None, norm_eps: float = 0.0,
+                   keys_as_values: bool = False, q_maps: int = 1) -> torch.Tensor:
     """Prepares attention whose projections carry biases and whose heads are rotated in part: ``qkv`` [T, >= nq dk +
     nkv dk + nkv dv] (float32, the stacked product; further columns are left alone; ``kv_heads`` 0 for queries only)
-    gets its biases, columns [rot_offset, rot_offset + rot_dims) of every query and key head are rotated (column i of
+    gets its biases, every query / key head its RMS norm where ``q_norm`` / ``k_norm`` [dk] is given (``norm_eps`` inside
+    the root, one weight for all heads), columns [rot_offset, rot_offset + rot_dims) of every query and key head are rotated (column i of
     the first half with column i + rot_dims / 2, by position * inv_freq[i], cosine and sine times ``rot_amplitude``), query head h is multiplied by
     ``q_factor[h]``, keys and values go to the token's page row in ``cache`` [pages, 2, nkv, page, pad_dim], and the
-    queries come back as [T, nq, pad_dim] in ``out_dtype`` with zero columns beyond dk."""
-    _need_cuda(qkv, q_bias, k_bias, v_bias, q_factor, inv_freq, cache, block_table, request_of_token, positions)
+    queries come back as [T, nq, pad_dim] in ``out_dtype`` with zero columns beyond dk.  ``keys_as_values``: the product
+    has no value columns, a head's value row is its key as projected, ahead of norm and rotation.  ``q_maps`` m > 1: a
+    head's dk columns are m queries side by side, over keys that lie side by side in the same way; the queries come back
+    as [T, nq * m, pad_dim], each in its own columns of the row and zero elsewhere."""
+    _need_cuda(qkv, q_bias, k_bias, v_bias, q_factor, inv_freq, q_norm, k_norm, cache, block_table, request_of_token, positions)
     assert qkv.dtype == torch.float32 and qkv.dim() == 2 and qkv.stride(1) == 1
-    assert qkv.shape[1] >= q_heads * key_dim + kv_heads * (key_dim + value_dim)
-    for t, n in ((q_bias, q_heads * key_dim), (k_bias, kv_heads * key_dim), (v_bias, kv_heads * value_dim),
+    assert qkv.shape[1] >= q_heads * key_dim + kv_heads * (key_dim + (0 if keys_as_values else value_dim))
+    for t, n in ((q_norm, key_dim), (k_norm, key_dim), (q_bias, q_heads * key_dim), (k_bias, kv_heads * key_dim), (v_bias, kv_heads * value_dim),
                  (q_factor, q_heads), (inv_freq, rot_dims // 2)):
         assert t is None or (t.dtype == torch.float32 and t.numel() == n and t.is_contiguous())
     num_pages, page_size = 0, 1
@@ -541,13 +560,25 @@ def qkv_rope_write(qkv: torch.Tensor, q_heads: int, kv_heads: int, key_dim: int,
         num_pages, c_heads, page_size, c_dim = _cache_dims(cache)
         assert (c_heads, c_dim) == (kv_heads, pad_dim) and cache.dtype == out_dtype
     tokens = qkv.shape[0]
-    q_out = torch.empty((tokens, q_heads, pad_dim), dtype=out_dtype, device=qkv.device)
+    q_out = torch.empty((tokens, q_heads * q_maps, pad_dim), dtype=out_dtype, device=qkv.device)
     _call(f"kirai_qkv_rope_write_{_suffix(out_dtype)}", _ptr(qkv), _l(qkv.stride(0)), _ptr(q_bias), _ptr(k_bias), _ptr(v_bias),
-          _ptr(q_factor), _ptr(inv_freq if rot_dims else None), _i(rot_offset), _i(rot_dims), _f(rot_amplitude), _ptr(q_out),
+          _ptr(q_factor), _ptr(q_norm), _ptr(k_norm), _f(norm_eps), _ptr(inv_freq if rot_dims else None), _i(rot_offset), _i(rot_dims), _f(rot_amplitude), _ptr(q_out),
           _ptr(cache if kv_heads else None), _ptr(block_table), _ptr(request_of_token), _ptr(positions), _i(tokens),
-          _i(q_heads), _i(kv_heads), _i(key_dim), _i(value_dim), _i(pad_dim), _i(page_size), _i(block_table.shape[1]),
-          _i(num_pages), _ptr(error_flag(qkv.device)), _stream())
+          _i(q_heads), _i(kv_heads), _i(key_dim), _i(value_dim), _i(pad_dim), _i(q_maps), _i(int(keys_as_values)), _i(page_size),
+          _i(block_table.shape[1]), _i(num_pages), _ptr(error_flag(qkv.device)), _stream())
     return q_out
+
+
+def map_difference(x: torch.Tensor, heads: int, used: int, pad_dim: int, factor: float, eps: float, out_factor: float) -> torch.Tensor:
+    """Two attention maps over the same values made one: ``x`` [T, heads * 2 * pad_dim] (a head's two outputs side by side,
+    the first ``used`` columns of each); o = first - ``factor`` * second, divided per head by its root mean square
+    (``eps`` inside the root), times ``out_factor``; returns [T, heads * used]."""
+    _need_cuda(x)
+    assert x.dim() == 2 and x.is_contiguous() and x.shape[1] == heads * 2 * pad_dim
+    out = torch.empty((x.shape[0], heads * used), dtype=x.dtype, device=x.device)
+    _call(f"kirai_map_difference_{_suffix(x.dtype)}", _ptr(x), _ptr(out), _i(x.shape[0]), _i(heads), _i(used), _i(pad_dim), _f(factor),
+          _f(eps), _f(out_factor), _stream())
+    return out
 
 
 def latent_prepare(down: torch.Tensor, q_rank: int, kv_rank: int, rot_dims: int, q_weight: Optional[torch.Tensor],
@@ -671,23 +702,123 @@ def gated_group_norm(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, 
     return out
 
 
-def conv_silu(x: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, conv_offset: int,
-              batch) -> torch.Tensor:
-    """Causal convolution per channel with silu over each request's tokens of this step.  ``x`` [T, C] (float32, a
-    run of columns of a wider tensor is allowed); ``taps`` [C, K] (float32), whose last column weighs the token
+def conv_rows(x: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, conv_offset: int,
+              batch, silu: bool = False, in_bias: Optional[torch.Tensor] = None, pair_block: int = 0, pair_tokens: int = 0):
+    """Causal convolution per channel (with ``silu``: then silu) over each request's tokens of this step.  ``x`` [T, C]
+    (float32, a run of columns of a wider tensor is allowed), plus ``in_bias`` [C] on every row that enters; ``taps`` [C, K] (float32), whose last column weighs the token
     itself; the K - 1 rows before a request's first row of this step come from its slot of ``state`` [slots, L]
-    (float32) at columns [conv_offset, conv_offset + (K - 1) C), which afterwards hold the request's last K - 1 rows."""
-    _need_cuda(x, taps, bias, state)
+    (float32) at columns [conv_offset, conv_offset + (K - 1) C), which afterwards hold the request's last K - 1 rows (with
+    their bias; zeros lie before a sequence's start).  Returns [T, C] (float32); with ``pair_block`` b also the same rows
+    as two bfloat16 numbers each, [C / b, pair_tokens, 2 b]: per block of channels the values rounded, then what the
+    rounding left (rows beyond T are not written)."""
+    _need_cuda(x, taps, bias, state, in_bias)
     assert x.dtype == torch.float32 and x.dim() == 2 and x.stride(1) == 1
     channels, width = x.shape[1], taps.shape[1]
     assert taps.dtype == torch.float32 and taps.shape == (channels, width) and taps.is_contiguous()
-    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == channels and bias.is_contiguous())
+    for b in (bias, in_bias):
+        assert b is None or (b.dtype == torch.float32 and b.numel() == channels and b.is_contiguous())
     assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous()
     out = torch.empty((x.shape[0], channels), dtype=torch.float32, device=x.device)
-    _call("kirai_conv_silu", _ptr(x), _l(x.stride(0)), _ptr(taps), _ptr(bias), _ptr(state), _l(state.shape[1]), _l(conv_offset),
-          _ptr(batch.request_of_token), _ptr(batch.query_start), _ptr(batch.slots), _ptr(out), _i(x.shape[0]),
-          _i(batch.num_requests), _i(channels), _i(width), _i(state.shape[0]), _stream())
+    pair = None
+    if pair_block:
+        assert channels % pair_block == 0 and pair_tokens >= x.shape[0]
+        pair = torch.empty((channels // pair_block, pair_tokens, 2 * pair_block), dtype=torch.bfloat16, device=x.device)
+    _call("kirai_conv_rows", _ptr(x), _l(x.stride(0)), _ptr(taps), _ptr(in_bias), _ptr(bias), _ptr(state), _l(state.shape[1]),
+          _l(conv_offset), _ptr(batch.request_of_token), _ptr(batch.query_start), _ptr(batch.slots), _ptr(out), _ptr(pair),
+          _i(pair_block), _i(pair_tokens), _i(int(silu)), _i(x.shape[0]), _i(batch.num_requests), _i(channels), _i(width),
+          _i(state.shape[0]), _stream(), detail=f" c={channels}" if _timer is not None else "")
+    return (out, pair) if pair_block else out
+
+
+def conv_silu(x: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, conv_offset: int,
+              batch) -> torch.Tensor:
+    """``conv_rows`` with silu."""
+    return conv_rows(x, taps, bias, state, conv_offset, batch, silu=True)
+
+
+def block_product(u: torch.Tensor, weight: torch.Tensor, blocks: int) -> torch.Tensor:
+    """A product per block of channels in 32-bit multiply-adds: ``u`` [T, blocks * b] (float32), ``weight`` [blocks, N, b]
+    (float32); returns [T, blocks * N] (float32)."""
+    return head_linear_gate(u, weight, blocks, u.shape[1] // blocks)
+
+
+def block_product_pairs(pair: torch.Tensor, weight) -> torch.Tensor:
+    """The same on the tensor cores without rounding ``u`` to 16 bits: ``pair`` [blocks, P, 2 b] (what ``conv_rows`` left, P
+    a multiple of 128) times ``weight`` [blocks * N, 2 b] (bfloat16, every row twice side by side); returns [blocks, P, N]
+    (float32, 32-bit accumulation)."""
+    blocks, tokens, cols = pair.shape
+    assert tokens % 128 == 0
+    y = linear_grouped(pair.view(blocks * tokens, cols), weight, blocks, _block_tiles(pair.device, blocks, tokens), out_dtype=torch.float32)
+    return y.view(blocks, tokens, -1)
+
+
+def real_gated_scan(u: torch.Tensor, gates: torch.Tensor, block: int, branch: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor,
+                    branch_bias: torch.Tensor, rate: torch.Tensor, state: torch.Tensor, state_offset: int, batch, out: torch.Tensor,
+                    factor: float = 1.0) -> torch.Tensor:
+    """The real-gated linear recurrence over each request's tokens of this step, per channel: r and i are the sigmoids of
+    the gates' pre-activations plus their biases, a = exp(rate * r), S <- a S + sqrt(1 - a^2) i u, S in the request's
+    slot of ``state`` [slots, L] (float32) from column ``state_offset``; ``out`` [T, C] (a run of columns of a wider
+    buffer is allowed) receives factor * S * gelu_tanh(branch + branch_bias) in its own dtype.  ``u`` [T, C]; ``gates``
+    [T, blocks * 2 block] or [blocks, P, 2 block]: per block of channels the r's, then the i's; ``branch`` [T, C] (a run of
+    columns is allowed); all float32."""
+    _need_cuda(u, gates, branch, r_bias, i_bias, branch_bias, rate, state, out)
+    tokens, channels = u.shape
+    blocks = channels // block
+    for t in (u, gates, branch, state, r_bias, i_bias, branch_bias, rate):
+        assert t.dtype == torch.float32
+    assert u.is_contiguous() and gates.is_contiguous() and blocks * block == channels
+    for t in (r_bias, i_bias, branch_bias, rate):
+        assert t.numel() == channels and t.is_contiguous()
+    if gates.dim() == 3:
+        assert gates.shape[0] == blocks and gates.shape[1] >= tokens and gates.shape[2] == 2 * block
+        gate_token, gate_block = 2 * block, gates.shape[1] * 2 * block
+    else:
+        assert gates.shape == (tokens, 2 * channels)
+        gate_token, gate_block = 2 * channels, 2 * block
+    assert branch.shape == (tokens, channels) and branch.stride(1) == 1 and out.shape == (tokens, channels) and out.stride(1) == 1
+    assert state.dim() == 2 and state.is_contiguous()
+    _call(f"kirai_real_gated_scan_{_suffix(out.dtype)}", _ptr(u), _ptr(gates), _l(gate_token), _l(gate_block), _i(block), _ptr(branch),
+          _l(branch.stride(0)), _ptr(r_bias), _ptr(i_bias), _ptr(branch_bias), _ptr(rate), _f(factor), _ptr(state), _l(state.shape[1]),
+          _l(state_offset), _ptr(batch.query_start), _ptr(batch.slots), _ptr(out), _l(out.stride(0)), _i(batch.num_requests),
+          _i(batch.max_query_len), _i(channels), _i(state.shape[0]), _stream())
     return out
+
+
+def streams_norm(streams: torch.Tensor, copies: int, update: Optional[tuple], read: Optional[torch.Tensor], weight: Optional[torch.Tensor],
+                 eps: float, out_dtype: torch.dtype, row_index: Optional[torch.Tensor] = None):
+    """A stream of ``copies`` copies read through a norm, after the update that the sub-layer before left: ``streams`` is
+    [T, copies, W], or [T, W] where all copies are still equal (both float32).  ``update`` = (y [T, W] float32, mix
+    [copies (from), copies (to)], add [copies]): copy t <- sum_f mix[f, t] copy f + add[t] y.  Then u = sum_t read[t] copy t
+    (None: their sum) leaves divided by its root mean square (``eps`` inside the root) times ``weight`` [W] in ``out_dtype``,
+    or as it is where ``weight`` is None (float32).  Returns (rows, streams after the update); the streams are updated in
+    place once they are [T, copies, W].  With ``row_index`` only those rows are produced and the streams are left as they
+    are."""
+    _need_cuda(streams, read, weight, row_index)
+    assert streams.dtype == torch.float32 and streams.is_contiguous() and streams.dim() in (2, 3)
+    tokens, width = streams.shape[0], streams.shape[-1]
+    equal = streams.dim() == 2
+    assert equal or streams.shape[1] == copies
+    y = mix = add = None
+    after = streams
+    if update is not None:
+        y, mix, add = update
+        _need_cuda(y, mix, add)
+        assert y.dtype == torch.float32 and y.shape == (tokens, width) and y.is_contiguous()
+        assert mix.dtype == torch.float32 and mix.shape == (copies, copies) and mix.is_contiguous()
+        assert add.dtype == torch.float32 and add.shape == (copies,) and add.is_contiguous()
+        if equal and row_index is None:
+            after = torch.empty((tokens, copies, width), dtype=torch.float32, device=streams.device)
+    assert read is None or (read.dtype == torch.float32 and read.shape == (copies,) and read.is_contiguous())
+    assert weight is None or (weight.dtype == torch.float32 and weight.numel() == width and weight.is_contiguous())
+    if row_index is not None:
+        assert row_index.dtype == torch.int32 and row_index.is_contiguous()
+    rows = tokens if row_index is None else row_index.numel()
+    out = torch.empty((rows, width), dtype=torch.float32 if weight is None else out_dtype, device=streams.device)
+    _call(f"kirai_streams_norm_{_suffix(out.dtype)}", _ptr(streams), _l(width if equal else copies * width), _l(0 if equal else width),
+          _ptr(after if update is not None and row_index is None else None), _ptr(y), _ptr(mix), _ptr(add), _ptr(read), _ptr(weight),
+          _ptr(out), _ptr(row_index), _i(rows), _i(copies), _i(width), _f(eps), _stream(),
+          detail=f" {'read' if y is None else 'update'}{' rows' if row_index is not None else ''}{' first' if equal else ''}" if _timer is not None else "")
+    return out, after
 
 
 STATE_WALK_LIMIT = 8  # steps whose longest run of tokens is at most this walk a matrix state token by token
@@ -778,15 +909,19 @@ def matrix_memory_walk(rows: torch.Tensor, in_bias: Optional[torch.Tensor], keep
     return o
 
 
-def head_gate_(x: torch.Tensor, gate: torch.Tensor, heads: int, used: int, pad_dim: int) -> torch.Tensor:
-    """``x`` [T, heads * pad_dim] (in place): the first ``used`` columns of head h times sigmoid(gate[t, h]); ``gate``
-    [T, heads] (float32; a run of columns of a wider product is allowed)."""
-    _need_cuda(x, gate)
+def head_gate_(x: torch.Tensor, gate: torch.Tensor, heads: int, used: int, pad_dim: int, out: Optional[torch.Tensor] = None,
+               factor: float = 1.0) -> torch.Tensor:
+    """``x`` [T, heads * pad_dim] (in place): the first ``used`` columns of head h times ``factor`` * sigmoid(gate[t, h]);
+    ``gate`` [T, heads] (float32; a run of columns of a wider product is allowed).  With ``out`` (the shape and dtype of
+    ``x``; a run of columns of a wider buffer is allowed) the rows go there, zero beyond ``used``, and ``x`` stays."""
+    _need_cuda(x, gate, out)
+    out = x if out is None else out
+    assert out.shape == x.shape and out.dtype == x.dtype and out.stride(1) == 1
     assert x.dim() == 2 and x.is_contiguous() and x.shape[1] == heads * pad_dim
     assert gate.dtype == torch.float32 and gate.dim() == 2 and gate.stride(1) == 1 and gate.shape == (x.shape[0], heads)
-    _call(f"kirai_head_gate_{_suffix(x.dtype)}", _ptr(x), _ptr(gate), _l(gate.stride(0)), _i(x.shape[0]), _i(heads), _i(used),
-          _i(pad_dim), _stream())
-    return x
+    _call(f"kirai_head_gate_{_suffix(x.dtype)}", _ptr(x), _ptr(gate), _l(gate.stride(0)), _ptr(out), _l(out.stride(0)), _i(x.shape[0]),
+          _i(heads), _i(used), _i(pad_dim), _f(factor), _stream())
+    return out
 
 
 def softcap_(x: torch.Tensor, cap: float) -> torch.Tensor:
@@ -1053,8 +1188,13 @@ def _attention_detail(q_heads: int, kv_heads: int, head_dim: int, window: Option
     return f" heads={q_heads} kv={kv_heads} d={head_dim} mask={mask_code(window, chunk, keep_first)}"
 
 
-def _capped(name: str, softcap: Optional[float]):
-    """The entry point ``name`` or its form with a soft cap on the scores, and that form's extra argument."""
+def _capped(name: str, softcap: Optional[float], sinks: Optional[torch.Tensor] = None, q_heads: int = 0):
+    """The entry point ``name`` or its form with a soft cap on the scores or with a sink per query head (a score that
+    stands in the softmax's denominator and has no value; ``sinks`` [q_heads], float32), and that form's extra arguments."""
+    if sinks is not None:
+        _need_cuda(sinks)
+        assert sinks.dtype == torch.float32 and sinks.numel() == q_heads and sinks.is_contiguous()
+        return name.replace("_bf16", "_sink_bf16").replace("_f32", "_sink_f32"), (_f(softcap or 0.0), _ptr(sinks))
     if softcap:
         return name.replace("_bf16", "_softcap_bf16").replace("_f32", "_softcap_f32"), (_f(softcap),)
     return name, ()
@@ -1062,7 +1202,8 @@ def _capped(name: str, softcap: Optional[float]):
 
 def paged_attention_plain(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
                           request_of_token: torch.Tensor, positions: torch.Tensor, window: Optional[int],
-                          scale: float, chunk: Optional[int] = None, softcap: Optional[float] = None, keep_first: int = 0) -> torch.Tensor:
+                          scale: float, chunk: Optional[int] = None, softcap: Optional[float] = None, keep_first: int = 0,
+                          sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal grouped-query attention of ``q`` [T, nq, d] over the paged cache; returns [T, nq * d].  ``chunk``: a
     query sees the keys of its own chunk of that many positions only; ``softcap`` c: scores become c tanh(score / c)."""
     _need_cuda(q, cache, block_table, request_of_token, positions)
@@ -1070,7 +1211,7 @@ def paged_attention_plain(q: torch.Tensor, cache: torch.Tensor, block_table: tor
     rows, q_heads, qd, q_stride = _head_view(q)
     assert qd == head_dim and q.dtype == cache.dtype
     out = torch.empty((rows, q_heads * head_dim), dtype=q.dtype, device=q.device)
-    name, cap = _capped(f"kirai_paged_attention_plain_{_suffix(q.dtype)}", softcap)
+    name, cap = _capped(f"kirai_paged_attention_plain_{_suffix(q.dtype)}", softcap, sinks, q_heads)
     _call(name, _ptr(q), _ptr(cache), _ptr(out), _ptr(block_table),
           _ptr(request_of_token), _ptr(positions), _i(rows), _i(q_heads), _i(kv_heads), _i(head_dim), _l(q_stride),
           _i(page_size), _i(block_table.shape[1]), _i(num_pages), _i(mask_code(window, chunk, keep_first)), _f(scale), *cap,
@@ -1111,7 +1252,7 @@ def attention_prefill_takes_tcgen05(q_heads: int, kv_heads: int, head_dim: int, 
 def attention_prefill(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, query_start: torch.Tensor,
                       context_len: torch.Tensor, max_query_len: int, window: Optional[int], scale: float,
                       tcgen05: Optional[bool] = None, out: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
-                      softcap: Optional[float] = None, keep_first: int = 0) -> torch.Tensor:
+                      softcap: Optional[float] = None, keep_first: int = 0, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """bf16 tensor-core attention for runs of new tokens (prompt portions, or any mix): q [T, nq, d].
     ``query_start`` holds rows of ``q`` and of the result, so the requests given may be a part of a larger batch
     (``out`` is then the whole batch's result, of which only their rows are written).  ``tcgen05`` picks the kernel (None: the tcgen05 kernel where it takes the shape, else the
@@ -1127,7 +1268,7 @@ def attention_prefill(q: torch.Tensor, cache: torch.Tensor, block_table: torch.T
     if out is None:
         out = torch.empty((rows, q_heads * head_dim), dtype=q.dtype, device=q.device)
     assert out.shape == (rows, q_heads * head_dim) and out.dtype == q.dtype and out.is_contiguous()
-    name, cap = _capped("kirai_attention_prefill_tc_bf16" if tcgen05 else "kirai_attention_prefill_bf16", softcap)
+    name, cap = _capped("kirai_attention_prefill_tc_bf16" if tcgen05 else "kirai_attention_prefill_bf16", softcap, sinks, q_heads)
     _call(name, _ptr(q), _ptr(cache), _ptr(out),
           _ptr(block_table), _ptr(query_start), _ptr(context_len), _i(requests), _i(max_query_len), _i(q_heads), _i(kv_heads),
           _i(head_dim), _l(q_stride), _i(page_size), _i(block_table.shape[1]), _i(num_pages), _i(mask_code(window, chunk, keep_first)), _f(scale),
@@ -1225,7 +1366,8 @@ def decode_plan(context_lens, kv_heads: int, window: Optional[int] = None, tile:
 
 def attention_decode(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, context_len: torch.Tensor,
                      window: Optional[int], scale: float, num_splits: int = 1, out: Optional[torch.Tensor] = None,
-                     chunk: Optional[int] = None, softcap: Optional[float] = None, keep_first: int = 0) -> torch.Tensor:
+                     chunk: Optional[int] = None, softcap: Optional[float] = None, keep_first: int = 0,
+                     sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """bf16 tensor-core attention for a batch in which every request brings one token: q [R, nq, d] (row r of ``q``,
     of the tables and of the result belongs to request r; ``out`` may be the head of a larger result)."""
     _need_cuda(q, cache, block_table, context_len)
@@ -1240,7 +1382,7 @@ def attention_decode(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Te
     if num_splits > 1 and not decode_pair_merges(rows * kv_heads, num_splits, head_dim, decode_cluster_room(q.device, head_dim, q_heads // kv_heads), q_heads // kv_heads):
         # the ranges' results go through a buffer and a second kernel
         partial = torch.empty((rows, q_heads, num_splits, head_dim + 2), dtype=torch.float32, device=q.device)
-    name, cap = _capped("kirai_attention_decode_bf16", softcap)
+    name, cap = _capped("kirai_attention_decode_bf16", softcap, sinks, q_heads)
     _call(name, _ptr(q), _ptr(cache), _ptr(out), _ptr(partial), _ptr(block_table),
           _ptr(context_len), _i(rows), _i(q_heads), _i(kv_heads), _i(head_dim), _l(q_stride), _i(page_size),
           _i(block_table.shape[1]), _i(num_pages), _i(mask_code(window, chunk, keep_first)), _f(scale), *cap, _i(num_splits),
@@ -1261,7 +1403,8 @@ def sm_count(device: torch.device) -> int:
 def attention_decode_balanced(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, context_len: torch.Tensor,
                               window: Optional[int], scale: float, ctas: Optional[int] = None,
                               out: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
-                              softcap: Optional[float] = None, keep_first: int = 0) -> torch.Tensor:
+                              softcap: Optional[float] = None, keep_first: int = 0,
+                              sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The decode attention with the key tiles of all (request, kv head) pairs cut into ``ctas`` equal ranges
     (default: one per SM), so that every CTA reads the same number of keys whatever the batch looks like."""
     _need_cuda(q, cache, block_table, context_len)
@@ -1274,7 +1417,7 @@ def attention_decode_balanced(q: torch.Tensor, cache: torch.Tensor, block_table:
         out = torch.empty((rows, q_heads * head_dim), dtype=q.dtype, device=q.device)
     assert out.shape == (rows, q_heads * head_dim) and out.dtype == q.dtype and out.is_contiguous()
     partial = torch.empty((ctas, 2, 16, head_dim + 2), dtype=torch.float32, device=q.device)
-    name, cap = _capped("kirai_attention_decode_balanced_bf16", softcap)
+    name, cap = _capped("kirai_attention_decode_balanced_bf16", softcap, sinks, q_heads)
     _call(name, _ptr(q), _ptr(cache), _ptr(out), _ptr(partial), _ptr(block_table),
           _ptr(context_len), _i(rows), _i(q_heads), _i(kv_heads), _i(head_dim), _l(q_stride), _i(page_size),
           _i(block_table.shape[1]), _i(num_pages), _i(mask_code(window, chunk, keep_first)), _f(scale), *cap, _i(ctas),
@@ -1283,7 +1426,8 @@ def attention_decode_balanced(q: torch.Tensor, cache: torch.Tensor, block_table:
 
 
 def paged_attention(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, batch, window: Optional[int],
-                    scale: float, chunk: Optional[int] = None, softcap: Optional[float] = None, keep_first: int = 0) -> torch.Tensor:
+                    scale: float, chunk: Optional[int] = None, softcap: Optional[float] = None, keep_first: int = 0,
+                    sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of the product path over the paged cache for the tokens of ``batch``
     (a kirai_b200.engine.batch.StepBatch).  float32 takes the plain kernel; bfloat16 takes the
     tensor-core kernels (the decode kernel when every request brings one token), or the plain
@@ -1292,7 +1436,7 @@ def paged_attention(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Ten
     fast = attention_takes_tensor_cores(q.dtype, head_dim) and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
     if not fast:
         return paged_attention_plain(q, cache, block_table, batch.request_of_token, batch.positions, window, scale,
-                                     chunk, softcap, keep_first)
+                                     chunk, softcap, keep_first, sinks)
     decode_rows = batch.num_requests if batch.decode_only else getattr(batch, "num_decode", 0)
     if decode_rows and q_heads // kv_heads <= 16:
         # The requests that bring one token stand first in the batch (the batch builder puts them there) and take the
@@ -1300,20 +1444,22 @@ def paged_attention(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Ten
         # write their rows of one result.  A prompt kernel alone would give a decoding request one CTA per kv head.
         out = torch.empty((q.shape[0], q_heads * head_dim), dtype=q.dtype, device=q.device)
         _decode_rows(q[:decode_rows], cache, block_table[:decode_rows], batch, decode_rows, window, scale, out[:decode_rows],
-                     chunk, softcap, keep_first)
+                     chunk, softcap, keep_first, sinks)
         if decode_rows < batch.num_requests:
             attention_prefill(q, cache, block_table[decode_rows:], batch.query_start[decode_rows:], batch.context_len[decode_rows:],
-                              batch.max_query_len, window, scale, out=out, chunk=chunk, softcap=softcap, keep_first=keep_first)
+                              batch.max_query_len, window, scale, out=out, chunk=chunk, softcap=softcap, keep_first=keep_first,
+                              sinks=sinks)
         return out
     return attention_prefill(q, cache, block_table, batch.query_start, batch.context_len, batch.max_query_len, window, scale,
-                             chunk=chunk, softcap=softcap, keep_first=keep_first)
+                             chunk=chunk, softcap=softcap, keep_first=keep_first, sinks=sinks)
 
 
 def _decode_rows(q, cache, block_table, batch, rows: int, window: Optional[int], scale: float, out: torch.Tensor,
-                 chunk: Optional[int] = None, softcap: Optional[float] = None, keep_first: int = 0) -> None:
+                 chunk: Optional[int] = None, softcap: Optional[float] = None, keep_first: int = 0,
+                 sinks: Optional[torch.Tensor] = None) -> None:
     """The decode attention of the first ``rows`` requests of ``batch`` (one token each)."""
     kv_heads = cache.shape[2]
-    mask = dict(chunk=chunk, softcap=softcap, keep_first=keep_first)
+    mask = dict(chunk=chunk, softcap=softcap, keep_first=keep_first, sinks=sinks)
     if chunk:
         window = None
     reach = (window + keep_first if window else None) or chunk  # the most keys a token sees: what the launch is planned for
@@ -1528,7 +1674,7 @@ def _chain_workspace(device: torch.device) -> torch.Tensor:
 
 
 def _launch_product(item) -> None:
-    x, weight, out, n, k, width, splits, form, row_scale, resid, norm_weight, sumsq_out = item
+    x, weight, out, n, k, width, splits, form, row_scale, resid, norm_weight, sumsq_out, gate = item
     tiled = isinstance(weight, TiledWeight)
     if row_scale is not None:
         sumsq, count, eps = row_scale
@@ -1537,7 +1683,7 @@ def _launch_product(item) -> None:
         scale_args = (_ptr(None), _i(0), _f(1.0), _f(0.0))
     _launch("kirai_gemm_bf16_general", _ptr(x), _ptr(weight.boxes if tiled else weight), _i(tiled), _ptr(out), _i(x.shape[0]),
             _i(n), _i(k), _l(x.stride(0)), _l(width), _i(splits), _i(form), *scale_args,
-            _ptr(resid), _ptr(norm_weight), _ptr(sumsq_out), _ptr(error_flag(x.device)), _stream(),
+            _ptr(resid), _ptr(norm_weight), _ptr(sumsq_out), _f(gate[0]), _f(gate[1]), _ptr(error_flag(x.device)), _stream(),
             detail=f" m={x.shape[0]} n={n} k={k} form={form}" if _timer is not None else "")
 
 
@@ -1579,12 +1725,13 @@ def flush_products() -> None:
         _launch_product(item)
 
 
-def _gemm(x, weight, out, n: int, k: int, width: int, splits: int, form: int, row_scale, resid, norm_weight, sumsq_out):
+def _gemm(x, weight, out, n: int, k: int, width: int, splits: int, form: int, row_scale, resid, norm_weight, sumsq_out,
+          gate: tuple = (0.0, 1.0)):
     if row_scale is not None:
         sumsq = row_scale[0]
         assert sumsq.dtype == torch.float32 and sumsq.dim() == 2 and sumsq.shape[1] == x.shape[0] and sumsq.is_contiguous()
-    item = (x, weight, out, n, k, width, splits, form, row_scale, resid, norm_weight, sumsq_out)
-    if chaining() and isinstance(weight, TiledWeight) and x.shape[0] <= 64 and splits == 0 and form not in (4, 5):
+    item = (x, weight, out, n, k, width, splits, form, row_scale, resid, norm_weight, sumsq_out, gate)
+    if chaining() and isinstance(weight, TiledWeight) and x.shape[0] <= 64 and splits == 0 and form not in (4, 5, 7):
         if _pending and _pending[0][0].shape[0] != x.shape[0]:
             flush_products()
         _pending.append(item)
@@ -1610,13 +1757,14 @@ def _check_product(x, weight) -> tuple:
 
 def linear_tcgen05(x: torch.Tensor, weight, out_dtype: Optional[torch.dtype] = None,
                    splits: int = 0, swiglu: bool = False, row_scale: Optional[tuple] = None,
-                   gate_act: str = "silu", relu2: bool = False) -> torch.Tensor:
+                   gate_act: str = "silu", relu2: bool = False, gate_limit: float = 0.0, gate_slope: float = 1.0) -> torch.Tensor:
     """bf16 ``x`` [M, K] times ``weight`` [N, K] transposed on the tcgen05 tensor cores (32-bit accumulation).
 
     ``weight`` is a row-major tensor or a ``TiledWeight``.  K and the row stride of ``x`` must be multiples of 8
     (TMA reads rows in 16-byte units).  ``splits`` > 1 cuts K between the CTAs of a cluster (0: chosen from the
     shape, at most 4).  With ``swiglu`` the rows of ``weight`` are 8 gate rows, their 8 up rows, 8 gate rows, ...
-    and the result is silu(gate) * up, [M, N / 2] (``gate_act`` "gelu_tanh": the tanh form of gelu in place of silu).
+    and the result is silu(gate) * up, [M, N / 2] (``gate_act`` "gelu_tanh": the tanh form of gelu in place of silu;
+    "clamped": the clamped form of ``gated_activation`` with ``gate_limit`` and ``gate_slope``).
     ``row_scale`` = (sumsq [P, M] float32, count, eps) multiplies
     row m of the product by 1 / sqrt(sum_p sumsq[p, m] / count + eps): ``x`` then holds rows that an RMSNorm left
     unscaled.  ``relu2``: the result is relu(product)^2 (bfloat16).
@@ -1629,9 +1777,8 @@ def linear_tcgen05(x: torch.Tensor, weight, out_dtype: Optional[torch.dtype] = N
         assert out_dtype == torch.bfloat16
     width = n // 2 if swiglu else n
     out = torch.empty((m, width), dtype=out_dtype, device=x.device)
-    form = (5 if gate_act == "gelu_tanh" else 2) if swiglu else (4 if relu2 else (0 if out_dtype == torch.bfloat16 else 1))
-    assert gate_act in GATED_ACTIVATIONS
-    _gemm(x, weight, out, n, k, width, splits, form, row_scale, None, None, None)
+    form = {"silu": 2, "gelu_tanh": 5, "clamped": 7}[gate_act] if swiglu else (4 if relu2 else (0 if out_dtype == torch.bfloat16 else 1))
+    _gemm(x, weight, out, n, k, width, splits, form, row_scale, None, None, None, (float(gate_limit), float(gate_slope)))
     return out
 
 

@@ -4,8 +4,6 @@
 //     and the row leaves as tanh(alpha * x) * w + b; no statistics of the row are taken;
 //   * the mean of two sub-layers' outputs, each divided by its root mean square over the row and multiplied by a
 //     weight of its own (two mixers that read the same rows side by side);
-//   * a causal convolution over a few taps per channel with silu, whose last taps - 1 input rows are state of the
-//     request, and the kernel that moves that state on;
 //   * the state-space recurrence S <- exp(-exp(A) dt) S + dt B x^T, y = S^T C + D x, per head, as a walk over a
 //     request's tokens of the step;
 //   * the matrix memory with exponential gates: S <- keep S + take k v^T and a normaliser n <- keep n + take k under a
@@ -168,76 +166,6 @@ KIRAI_EXPORT int kirai_gated_group_norm_bf16(const float* y, long y_stride, cons
                                              float eps, void* out, int rows, int groups, int group_width, int mode,
                                              cudaStream_t stream) {
     return gated_group_norm_launch<bf16>(y, y_stride, gate, g_stride, weight, eps, out, rows, groups, group_width, mode, stream);
-}
-
-// -------------------------------------------------------------- causal convolution + silu
-// Blocks (token, run of channels).  in [T, channels] (float32, row stride in_stride): what the convolution reads; taps_w
-// [channels, taps], whose last column weighs the token itself; the rows before a request's first row of this step are
-// the request's `taps - 1` kept rows, state [slots, state_len] from column conv_off, [taps - 1, channels], the newest
-// last (zeros at a sequence's start).  out [T, channels] (float32) = silu(bias + sum_j w[c, j] * in[t - (taps - 1) + j, c]).
-__global__ void conv_silu_kernel(const float* __restrict__ in, long in_stride, const float* __restrict__ taps_w,
-                                 const float* __restrict__ bias, const float* __restrict__ state, long state_len, long conv_off,
-                                 const int* __restrict__ request_of_token, const int* __restrict__ query_start,
-                                 const int* __restrict__ slots, float* __restrict__ out, int channels, int taps, int num_slots) {
-    pdl_launch_dependents();
-    const long token = blockIdx.x;
-    const int request = request_of_token[token];
-    const long first = query_start[request];
-    const int slot = slots[request];
-    pdl_wait();
-    if (slot < 0 || slot >= num_slots) return;
-    const int local = (int)(token - first);
-    const float* kept = state + slot * state_len + conv_off;
-    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < channels; c += gridDim.y * blockDim.x) {
-        float acc = bias ? bias[c] : 0.0f;
-        for (int j = 0; j < taps; ++j) {
-            const int at = local - (taps - 1) + j;
-            const float v = at >= 0 ? in[(first + at) * in_stride + c] : kept[(long)(taps - 1 + at) * channels + c];
-            acc = fmaf(taps_w[(long)c * taps + j], v, acc);
-        }
-        out[token * channels + c] = sf_silu(acc);
-    }
-}
-
-// A thread per (request, channel): the kept rows become the last taps - 1 input rows of the request after this step.
-__global__ void conv_state_kernel(const float* __restrict__ in, long in_stride, float* __restrict__ state, long state_len,
-                                  long conv_off, const int* __restrict__ query_start, const int* __restrict__ slots, int requests,
-                                  int channels, int taps, int num_slots) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const long at = blockIdx.x * (long)blockDim.x + threadIdx.x;
-    if (at >= (long)requests * channels) return;
-    const int request = (int)(at / channels), c = (int)(at - (long)request * channels);
-    const int slot = slots[request];
-    if (slot < 0 || slot >= num_slots) return;
-    const long first = query_start[request];
-    const int count = (int)(query_start[request + 1] - first);
-    float* kept = state + slot * state_len + conv_off;
-    // ascending: entry k takes input row count - (taps - 1) + k, or the kept row count + k (> k, not yet overwritten)
-    for (int k = 0; k < taps - 1; ++k) {
-        const int src = count - (taps - 1) + k;
-        kept[(long)k * channels + c] = src >= 0 ? in[(first + src) * in_stride + c] : kept[(long)(count + k) * channels + c];
-    }
-}
-
-KIRAI_EXPORT int kirai_conv_silu(const float* in, long in_stride, const float* taps_w, const float* bias, float* state,
-                                 long state_len, long conv_off, const int* request_of_token, const int* query_start,
-                                 const int* slots, float* out, int tokens, int requests, int channels, int taps, int num_slots,
-                                 cudaStream_t stream) {
-    if (tokens <= 0) return 0;
-    if (channels <= 0 || taps <= 0 || requests <= 0 || conv_off < 0 || conv_off + (long)(taps - 1) * channels > state_len)
-        return KIRAI_ERR_BAD_SIZE;
-    const int threads = channels >= 1024 ? 256 : 128;
-    // few tokens: a token's channels spread over several blocks, so that a step of single tokens fills more of the device
-    int spread = 1;
-    while (spread < 16 && tokens * spread < 256 && threads * spread * 2 <= channels) spread *= 2;
-    int status = launch_pdl(conv_silu_kernel, dim3(tokens, spread), dim3(threads), 0, stream, 1u, in, in_stride, taps_w, bias,
-                            (const float*)state, state_len, conv_off, request_of_token, query_start, slots, out, channels, taps,
-                            num_slots);
-    if (status != 0 || taps == 1) return status;
-    const long units = (long)requests * channels;
-    return launch_pdl(conv_state_kernel, dim3((unsigned)((units + 255) / 256)), dim3(256), 0, stream, 1u, in, in_stride, state,
-                      state_len, conv_off, query_start, slots, requests, channels, taps, num_slots);
 }
 
 // ------------------------------------------------------------------ state-space walk
@@ -470,40 +398,77 @@ KIRAI_EXPORT int kirai_matrix_memory_walk(const float* rows, long row_stride, co
 }
 
 // ------------------------------------------------------------------ small element-wise steps
-// x [T, heads * dpad] (in place): the first `used` columns of head h times sigmoid(gate[t, h]) (float32, row stride).
+// x [T, heads * dpad]: the first `used` columns of head h times factor * sigmoid(gate[t, h]) (float32, row stride), written
+// to out (row stride out_stride; it may be x itself).  Into a buffer of its own every column is written, the padding as zeros.
 template <typename T>
-__global__ void head_gate_kernel(T* __restrict__ x, const float* __restrict__ gate, long gate_stride, long rows, int heads,
-                                 int used, int dpad) {
+__global__ void head_gate_kernel(const T* x, const float* __restrict__ gate, long gate_stride, T* out, long out_stride, long rows,
+                                 int heads, int used, int dpad, float factor) {
     pdl_launch_dependents();
     pdl_wait();
-    const long per_row = (long)heads * used, total = rows * per_row;
+    const bool in_place = x == out;
+    const int cols = in_place ? used : dpad;
+    const long per_row = (long)heads * cols, total = rows * per_row;
     for (long at = blockIdx.x * (long)blockDim.x + threadIdx.x; at < total; at += (long)gridDim.x * blockDim.x) {
         const long row = at / per_row;
         const int col = (int)(at - row * per_row);
-        const int head = col / used, c = col - head * used;
-        T* p = x + (row * heads + head) * dpad + c;
-        *p = from_f32<T>(to_f32<T>(*p) * sf_sigmoid(gate[row * gate_stride + head]));
+        const int head = col / cols, c = col - head * cols;
+        float v = 0.0f;
+        if (c < used) v = to_f32<T>(x[(row * heads + head) * dpad + c]) * (factor * sf_sigmoid(gate[row * gate_stride + head]));
+        out[row * out_stride + (long)head * dpad + c] = from_f32<T>(v);
+    }
+}
+
+// The same for bfloat16, eight columns a thread (every width, stride and pointer allows 16-byte accesses).
+__global__ void head_gate_vec_kernel(const bf16* x, const float* __restrict__ gate, long gate_stride, bf16* out, long out_stride,
+                                     long rows, int heads, int used, int dpad, float factor) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int pieces = dpad >> 3;
+    const long per_row = (long)heads * pieces, total = rows * per_row;
+    for (long at = blockIdx.x * (long)blockDim.x + threadIdx.x; at < total; at += (long)gridDim.x * blockDim.x) {
+        const long row = at / per_row;
+        const int piece = (int)(at - row * per_row);
+        const int head = piece / pieces, c = (piece - head * pieces) * 8;
+        uint4 packed = make_uint4(0u, 0u, 0u, 0u);
+        if (c < used) {
+            const float g = factor * sf_sigmoid(gate[row * gate_stride + head]);
+            packed = *reinterpret_cast<const uint4*>(x + (row * heads + head) * dpad + c);
+            __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float2 v = __bfloat1622float2(p[j]);
+                p[j] = __floats2bfloat162_rn(v.x * g, v.y * g);
+            }
+        }
+        *reinterpret_cast<uint4*>(out + row * out_stride + (long)head * dpad + c) = packed;
     }
 }
 
 template <typename T>
-static int head_gate_launch(void* x, const float* gate, long gate_stride, int rows, int heads, int used, int dpad,
-                            cudaStream_t stream) {
+static int head_gate_launch(const void* x, const float* gate, long gate_stride, void* out, long out_stride, int rows, int heads, int used,
+                            int dpad, float factor, cudaStream_t stream) {
     if (rows <= 0) return 0;
-    if (heads <= 0 || used <= 0 || dpad < used) return KIRAI_ERR_BAD_SIZE;
-    const long total = (long)rows * heads * used;
+    if (heads <= 0 || used <= 0 || dpad < used || out_stride < (long)heads * dpad || (x == out && out_stride != (long)heads * dpad))
+        return KIRAI_ERR_BAD_SIZE;
+    if (sizeof(T) == 2 && used % 8 == 0 && dpad % 8 == 0 && out_stride % 8 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0) {
+        const long pieces = (long)rows * heads * (dpad / 8);
+        const unsigned vec_blocks = (unsigned)min((pieces + 255) / 256, (long)148 * 16);
+        return launch_pdl(head_gate_vec_kernel, dim3(vec_blocks), dim3(256), 0, stream, 1u, (const bf16*)x, gate, gate_stride, (bf16*)out,
+                          out_stride, (long)rows, heads, used, dpad, factor);
+    }
+    const long total = (long)rows * heads * dpad;
     const unsigned blocks = (unsigned)min((total + 255) / 256, (long)148 * 16);
-    return launch_pdl(head_gate_kernel<T>, dim3(blocks), dim3(256), 0, stream, 1u, (T*)x, gate, gate_stride, (long)rows, heads, used,
-                      dpad);
+    return launch_pdl(head_gate_kernel<T>, dim3(blocks), dim3(256), 0, stream, 1u, (const T*)x, gate, gate_stride, (T*)out, out_stride,
+                      (long)rows, heads, used, dpad, factor);
 }
 
-KIRAI_EXPORT int kirai_head_gate_f32(void* x, const float* gate, long gate_stride, int rows, int heads, int used, int dpad,
-                                     cudaStream_t stream) {
-    return head_gate_launch<float>(x, gate, gate_stride, rows, heads, used, dpad, stream);
+KIRAI_EXPORT int kirai_head_gate_f32(const void* x, const float* gate, long gate_stride, void* out, long out_stride, int rows, int heads,
+                                     int used, int dpad, float factor, cudaStream_t stream) {
+    return head_gate_launch<float>(x, gate, gate_stride, out, out_stride, rows, heads, used, dpad, factor, stream);
 }
-KIRAI_EXPORT int kirai_head_gate_bf16(void* x, const float* gate, long gate_stride, int rows, int heads, int used, int dpad,
-                                      cudaStream_t stream) {
-    return head_gate_launch<bf16>(x, gate, gate_stride, rows, heads, used, dpad, stream);
+KIRAI_EXPORT int kirai_head_gate_bf16(const void* x, const float* gate, long gate_stride, void* out, long out_stride, int rows, int heads,
+                                      int used, int dpad, float factor, cudaStream_t stream) {
+    return head_gate_launch<bf16>(x, gate, gate_stride, out, out_stride, rows, heads, used, dpad, factor, stream);
 }
 
 // logits (float32, in place) <- cap * tanh(logits / cap)

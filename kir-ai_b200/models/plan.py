@@ -16,7 +16,7 @@ from typing import Dict, List, Optional
 
 import torch
 
-from ..parts.base import Norm, NormedSum, Runtime, ScaledSum, StreamCopy, WeightSpec
+from ..parts.base import Norm, NormedSum, Runtime, ScaledSum, StreamCopy, StreamUpdate, WeightSpec
 from ..parts.block import Block
 from ..parts.embedding import Embedding, OutputHead
 
@@ -143,7 +143,7 @@ class DecoderModel:
         return self
 
     def forward(self, batch, cache) -> tuple:
-        """The residual stream [T, H] (32-bit) and the last block's not-yet-added output."""
+        """The residual stream (32-bit; [T, H], or [T, copies, H] where the blocks keep several copies) and the last block's not-yet-added output."""
         nvtx = torch.cuda.nvtx if self.nvtx else None  # ranges around the layer calls, for a timeline tool
         with self.rt.ops.chained_products(self._kernels_only):
             embedding, order, delta = self.plan.embedding, self.plan.order, None
@@ -187,6 +187,10 @@ class DecoderModel:
         if isinstance(delta, ScaledSum) and not getattr(self.plan.final_norm, "takes_scaled_sum", False):
             self.rt.ops.add_scaled_into_residual(resid, delta.rows, delta.factor)
             delta = None
+        if isinstance(delta, StreamUpdate) and not getattr(self.plan.final_norm, "takes_streams", False):
+            # a norm of another kind reads the wanted rows' sums of the copies
+            resid, _ = self.rt.ops.streams_norm(resid, delta.mix.shape[0], delta.terms(), None, None, 0.0, torch.float32, row_index=rows)
+            rows, delta = torch.arange(resid.shape[0], dtype=torch.int32, device=resid.device), None
         with self.rt.ops.chained_products(self._kernels_only):
             normed = self.plan.final_norm.add_forward_rows(resid, delta, rows)
             logits = self.plan.head.forward(normed)

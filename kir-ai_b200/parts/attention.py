@@ -41,7 +41,10 @@ when i - j < W or j < F, so a sequence's first F keys stay visible at their true
 pages when the window gives the others back).  A ``RotaryEmbedding`` whose cosine and sine carry a factor
 (``amplitude``) is applied with it by the preparation kernel.  A ``RotaryEmbedding`` that pairs neighbouring columns
 has the rows of the q and k matrices (and biases) put in its ``head_order`` at load; scores do not change with the
-order of a head's columns, as long as queries and keys share it.
+order of a head's columns, as long as queries and keys share it.  A norm per head goes with these options too
+(the preparation kernel applies it ahead of the rotation).  ``keys_as_values``: there is no v matrix, a head's value is
+its key as projected, ahead of norm and rotation (keys and values are then cached side by side all the same).  ``sink`` s:
+every head's softmax has one more term exp(s) in its denominator that no value stands behind.
 """
 from __future__ import annotations
 
@@ -61,7 +64,8 @@ class GQAttention(Mixer):
                  names: Optional[Dict[str, str]] = None, value_dim: Optional[int] = None, bias: bool = False,
                  qk_norm_over: str = "head", out_dtype: Optional[torch.dtype] = None, head_factor: Optional[str] = None,
                  softcap: Optional[float] = None, chunk: Optional[int] = None, gate: Optional[str] = None,
-                 out_bias: Optional[str] = None, head_gate: Optional[str] = None, keep_first: int = 0):
+                 out_bias: Optional[str] = None, head_gate: Optional[str] = None, keep_first: int = 0,
+                 keys_as_values: bool = False, sink: Optional[float] = None):
         if q_heads % kv_heads:
             raise ValueError(f"{q_heads} query heads are not a multiple of {kv_heads} kv heads")
         if qk_norm_over not in ("head", "projection"):
@@ -97,12 +101,18 @@ class GQAttention(Mixer):
             raise ValueError("an output gate has a number per column or a number per head, not both")
         if (self.keep_first or head_gate) and reads_only:
             raise ValueError("kept first keys or a gate per head are not built for a layer that reads another layer's cache")
+        self.keys_as_values, self.sink, self.sinks = bool(keys_as_values), sink, None
+        if keys_as_values and (reads_only or self.value_dim != head_dim):
+            raise ValueError("values that are the keys as projected have the keys' width and need a layer with keys of its own")
+        if sink is not None and reads_only:
+            raise ValueError("a sink is not built for a layer that reads another layer's cache")
+        self.shares_products = False  # set by a mixer that makes this part's outer products itself
         self.out_bias_name = prefix + out_bias if out_bias else None
         self.head_factor = self.out_bias = None
         self.defer_output_bias = False  # a block whose next norm adds the bias sets this
         shifted_rotation = isinstance(position, RotaryEmbedding) and (position.offset != 0 or position.amplitude != 1.0
                                                                       or position.pairing != "halves")
-        self.wide = (head_gate is not None or self.keep_first > 0 or bias or self.value_dim != head_dim or (qk_norm_eps is not None and qk_norm_over == "projection")
+        self.wide = (keys_as_values or sink is not None or head_gate is not None or self.keep_first > 0 or bias or self.value_dim != head_dim or (qk_norm_eps is not None and qk_norm_over == "projection")
                      or head_factor is not None or gate is not None or shifted_rotation or self.softcap is not None
                      or self.chunk is not None or out_bias is not None)
         self.norm_over_projection = qk_norm_eps is not None and qk_norm_over == "projection"
@@ -113,12 +123,14 @@ class GQAttention(Mixer):
                                  "RotaryEmbedding or no position encoding, and none together with a norm over the projection")
             if self.norm_over_projection and (head_factor or gate):
                 raise ValueError("a head factor or an output gate is not built together with a norm over the projection")
-            if qk_norm_eps is not None and qk_norm_over == "head":
-                raise ValueError("a per-head q/k norm is not built together with biases or values of their own width")
+            if self.norm_over_projection and (keys_as_values or sink is not None):
+                raise ValueError("a norm over the projection is not built together with values that are the keys, or with a sink")
             self.pad_dim = -(-max(head_dim, self.value_dim) // 8) * 8
         sources = [(prefix + n["q"], q_heads * head_dim)]
         if not reads_only:
-            sources += [(prefix + n["k"], kv_heads * head_dim), (prefix + n["v"], kv_heads * self.value_dim)]
+            sources.append((prefix + n["k"], kv_heads * head_dim))
+            if not keys_as_values:
+                sources.append((prefix + n["v"], kv_heads * self.value_dim))
         if self.gate_name:
             sources.append((self.gate_name, q_heads * self.value_dim))
         if self.head_gate_name:
@@ -136,6 +148,7 @@ class GQAttention(Mixer):
             stacked_order[: q_heads * head_dim] = self.q_order
             if self.k_order is not None:
                 stacked_order[q_heads * head_dim : (q_heads + kv_heads) * head_dim] = q_heads * head_dim + self.k_order
+        self.sources, self.names = sources, {key: prefix + value for key, value in n.items()}
         self.qkv = Linear(sources, hidden_size, row_order=stacked_order)
         self.out = Linear([(prefix + n["o"], hidden_size)], q_heads * self.value_dim,
                           column_groups=(q_heads, self.value_dim, self.pad_dim) if self.wide else None)
@@ -161,7 +174,7 @@ class GQAttention(Mixer):
         return self.position is None or bool(self.position.kernels_only)
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
-        specs = {**self.qkv.weight_specs(), **self.out.weight_specs()}
+        specs = {} if self.shares_products else {**self.qkv.weight_specs(), **self.out.weight_specs()}
         if self.qk_norm_eps is not None:
             over = (self.q_heads, self.kv_heads) if self.norm_over_projection else (1, 1)
             specs[self.q_norm_name] = WeightSpec((over[0] * self.head_dim,), "norm")
@@ -171,7 +184,8 @@ class GQAttention(Mixer):
             specs[self.bias_names[0]] = WeightSpec((self.q_heads * self.head_dim,), "bias")
             if not self.reads_only:
                 specs[self.bias_names[1]] = WeightSpec((self.kv_heads * self.head_dim,), "bias")
-                specs[self.bias_names[2]] = WeightSpec((self.kv_heads * self.value_dim,), "bias")
+                if not self.keys_as_values:
+                    specs[self.bias_names[2]] = WeightSpec((self.kv_heads * self.value_dim,), "bias")
         if self.head_factor_name:
             specs[self.head_factor_name] = WeightSpec((self.q_heads,), "norm")
         if self.out_bias_name:
@@ -182,8 +196,11 @@ class GQAttention(Mixer):
 
     def load(self, weights, rt: Runtime) -> None:
         self.rt = rt
-        self.qkv.load(weights, rt)
-        self.out.load(weights, rt)
+        if not self.shares_products:
+            self.qkv.load(weights, rt)
+            self.out.load(weights, rt)
+        if self.sink is not None:
+            self.sinks = torch.full((self.q_heads,), float(self.sink), dtype=torch.float32, device=rt.device)
         if self.qk_norm_eps is not None:
             self.q_norm_weight = weights.on_device(self.q_norm_name, torch.float32)
             if not self.reads_only:
@@ -196,7 +213,8 @@ class GQAttention(Mixer):
                 self.k_bias = weights.on_device(self.bias_names[1], torch.float32)
                 if self.k_order is not None:
                     self.k_bias = self.k_bias[self.k_order.to(rt.device)].contiguous()
-                self.v_bias = weights.on_device(self.bias_names[2], torch.float32)
+                if not self.keys_as_values:
+                    self.v_bias = weights.on_device(self.bias_names[2], torch.float32)
         if self.head_factor_name:
             self.head_factor = weights.on_device(self.head_factor_name, torch.float32)
         if self.out_bias_name:
@@ -230,24 +248,53 @@ class GQAttention(Mixer):
         table = batch.block_tables[cache.group]
         qkv = self.qkv.forward(x, torch.float32)
         if not self.norm_over_projection:
-            rot = self.position
-            q = ops.qkv_rope_write(qkv, self.q_heads, nkv, self.head_dim, self.value_dim, self.pad_dim, self.q_bias, self.k_bias,
-                                   self.v_bias, self.head_factor, rot.inv_freq if rot is not None else None,
-                                   rot.offset if rot is not None else 0, rot.rotary_dim if rot is not None else 0,
-                                   cache.kv, table, batch.request_of_token, batch.positions, self.rt.dtype,
-                                   rot_amplitude=rot.amplitude if rot is not None else 1.0)
-            mixed = ops.paged_attention(q, cache.kv, table, batch, self.window, self.scale, chunk=self.chunk, softcap=self.softcap,
-                                        keep_first=self.keep_first)
-            gate_at = self.q_heads * self.head_dim + nkv * (self.head_dim + self.value_dim)
-            if self.gate_name:
-                ops.sigmoid_gate_(mixed, qkv[:, gate_at:], self.q_heads, self.value_dim, self.pad_dim)
-            if self.head_gate_name:
-                ops.head_gate_(mixed, qkv[:, gate_at : gate_at + self.q_heads], self.q_heads, self.value_dim, self.pad_dim)
-            return mixed
+            return self._mix_prepared(qkv, batch, cache)
         q = ops.qkv_wide_norm_write(qkv, self.q_heads, nkv, self.head_dim, self.value_dim, self.pad_dim, self.q_bias,
                                     self.k_bias, self.v_bias, self.q_norm_weight, self.k_norm_weight, self.qk_norm_eps or 0.0,
                                     cache.kv, table, batch.request_of_token, batch.positions, self.rt.dtype)
         return ops.paged_attention(q, cache.kv, table, batch, self.window, self.scale)
+
+    def _mix_prepared(self, qkv, batch, cache, out: Optional[torch.Tensor] = None, factor: float = 1.0) -> torch.Tensor:
+        """From the stacked product's 32-bit rows to what the output projection reads; a gate per head may write it into
+        ``out`` times ``factor``."""
+        ops = self.rt.ops
+        nkv = 0 if self.reads_only else self.kv_heads
+        table = batch.block_tables[cache.group]
+        rot = self.position
+        q = ops.qkv_rope_write(qkv, self.q_heads, nkv, self.head_dim, self.value_dim, self.pad_dim, self.q_bias, self.k_bias,
+                               self.v_bias, self.head_factor, rot.inv_freq if rot is not None else None,
+                               rot.offset if rot is not None else 0, rot.rotary_dim if rot is not None else 0,
+                               cache.kv, table, batch.request_of_token, batch.positions, self.rt.dtype,
+                               rot_amplitude=rot.amplitude if rot is not None else 1.0,
+                               q_norm=self.q_norm_weight, k_norm=self.k_norm_weight, norm_eps=self.qk_norm_eps or 0.0,
+                               keys_as_values=self.keys_as_values)
+        mixed = ops.paged_attention(q, cache.kv, table, batch, self.window, self.scale, chunk=self.chunk, softcap=self.softcap,
+                                    keep_first=self.keep_first, sinks=self.sinks)
+        gate_at = self.q_heads * self.head_dim + nkv * (self.head_dim + (0 if self.keys_as_values else self.value_dim))
+        if self.gate_name:
+            ops.sigmoid_gate_(mixed, qkv[:, gate_at:], self.q_heads, self.value_dim, self.pad_dim)
+        if self.head_gate_name:
+            return ops.head_gate_(mixed, qkv[:, gate_at : gate_at + self.q_heads], self.q_heads, self.value_dim, self.pad_dim,
+                                  out=out, factor=factor)
+        return mixed
+
+    # what a mixer that shares its products with another's needs (``parts.side_by_side.ScaledPairMixer``)
+    def can_share_products(self) -> bool:
+        """Whether another mixer may make this layer's outer products: a gate per head then writes what the output
+        projection reads, and no norm runs over the projection."""
+        return bool(self.wide and self.head_gate_name and not self.norm_over_projection and not self.gate_name and not self.reads_only
+                    and self.out_bias_name is None and self.q_order is None)
+
+    def input_sources(self):
+        return list(self.sources)
+
+    def output_source(self):
+        return self.names["o"], self.q_heads * self.value_dim, (self.q_heads, self.value_dim, self.pad_dim)
+
+    def mix_into(self, rows, batch, cache, out: torch.Tensor, factor: float = 1.0) -> torch.Tensor:
+        """Everything between the products: ``rows`` (float32, what the input matrices made) to ``out`` [T, q_heads *
+        pad_dim], what the output projection reads, times ``factor``."""
+        return self._mix_prepared(rows, batch, cache, out, factor)
 
     def forward_into_norm(self, x, batch, cache, write_cache, resid, spec):
         return self.out.forward_into_norm(self._mix(x, batch, cache, write_cache), resid, spec)

@@ -26,8 +26,8 @@ class WeightSpec:
     """Shape and role of one named tensor.  The role tells the random-weights
     mode how to fill it and the loader which dtype family it must have:
     ``linear`` and ``embedding`` are floating matrices, ``norm`` a floating
-    vector around one, ``bias`` a floating vector around zero, ``int_table`` an
-    integer table (kept as int32)."""
+    vector around one, ``bias`` a floating vector around zero, ``identity`` a square matrix
+    around the identity, ``int_table`` an integer table (kept as int32)."""
 
     shape: Tuple[int, ...]
     role: str = "linear"
@@ -115,6 +115,20 @@ class NormedSum:
     def settle(self, resid: torch.Tensor, ops, copy_dtype: Optional[torch.dtype] = None):
         """resid += norm(rows) in place; returns the stream's copy in ``copy_dtype`` when that is asked for."""
         return ops.norm_add(resid, self.rows, self.weight, self.eps, copy_dtype)
+
+
+@dataclass
+class StreamUpdate:
+    """What a sub-layer leaves when the stream is kept as several copies (``parts.streams``): from its output ``rows``
+    (float32 [T, width]) every copy is made afresh, copy t <- sum_f mix[f, t] copy f + add[t] * rows.  Whoever reads the
+    stream next makes the update in its own pass."""
+
+    rows: torch.Tensor
+    mix: torch.Tensor
+    add: torch.Tensor
+
+    def terms(self) -> tuple:
+        return (self.rows, self.mix, self.add)
 
 
 class Runtime:

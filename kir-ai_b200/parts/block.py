@@ -29,6 +29,11 @@ that reads the stream next are one pass over the row: the block hands what is le
 a norm that ``takes_normed_sum`` adds while it norms (the next sub-layer's, the next block's first, or the model's
 last); any other reader has it settled into the stream first.
 
+``streams`` keeps the stream as several copies (``parts.streams``): around each sub-layer a connection (``connection1``,
+``connection2``) says what the sub-layer reads of the copies, through its norm, and how the copies are made afresh from the
+old ones and the sub-layer's 32-bit output.  That update travels on as a ``StreamUpdate``, and the next reader (the next
+sub-layer's norm, the next block's first, or the model's last) makes it in its own pass.
+
 ``residual_scale`` m (``pre_norm`` only) multiplies what every sub-layer adds: h <- h + m * mixer(norm1(h)), then
 h <- h + m * ffn(norm2(h)).  The sub-layers then leave 32-bit rows (a feed-forward may leave several terms,
 ``FeedForward.forward_terms``), which travel to the next norm as a ``ScaledSum``; a norm that ``takes_scaled_sum`` adds
@@ -41,9 +46,9 @@ from typing import Dict, Optional, Tuple
 
 import torch
 
-from .base import FeedForward, FusedNormSpec, Mixer, Norm, NormedSum, Part, Runtime, ScaledSum, StreamCopy, UnscaledNorm, WeightSpec
+from .base import FeedForward, FusedNormSpec, Mixer, Norm, NormedSum, Part, Runtime, ScaledSum, StreamCopy, StreamUpdate, UnscaledNorm, WeightSpec
 
-ARRANGEMENTS = ("pre_norm", "parallel", "out_norm", "sandwich")
+ARRANGEMENTS = ("pre_norm", "parallel", "out_norm", "sandwich", "streams")
 
 
 def _offers(part, method: str, rows: int) -> bool:
@@ -56,7 +61,12 @@ def _offers(part, method: str, rows: int) -> bool:
 class Block(Part):
     def __init__(self, norm1: Norm, mixer: Mixer, norm2: Optional[Norm], ffn: Optional[FeedForward], arrangement: str = "pre_norm",
                  shift: Optional[Part] = None, residual_scale: Optional[float] = None, post_norm1: Optional[Norm] = None,
-                 post_norm2: Optional[Norm] = None):
+                 post_norm2: Optional[Norm] = None, connection1: Optional[Part] = None, connection2: Optional[Part] = None):
+        if (arrangement == "streams") != (connection1 is not None) or (connection2 is not None) != (arrangement == "streams" and ffn is not None):
+            raise ValueError("the streams arrangement, and it alone, has a connection around every sub-layer")
+        if arrangement == "streams" and ((ffn is None) != (norm2 is None) or shift is not None):
+            raise ValueError("the streams arrangement has its second norm exactly when it has a feed-forward, and no token shift")
+        self.connection1, self.connection2 = connection1, connection2
         if (arrangement == "sandwich") != (post_norm1 is not None) or (post_norm2 is not None) != (arrangement == "sandwich" and ffn is not None):
             raise ValueError("the sandwich arrangement, and it alone, has a norm on every sub-layer's output")
         if arrangement == "sandwich" and ((ffn is None) != (norm2 is None) or shift is not None):
@@ -84,7 +94,8 @@ class Block(Part):
             mixer.defer_output_bias = True
 
     def _parts(self):
-        return [p for p in (self.norm1, self.shift, self.mixer, self.post_norm1, self.norm2, self.ffn, self.post_norm2) if p is not None]
+        return [p for p in (self.norm1, self.connection1, self.shift, self.mixer, self.post_norm1, self.norm2, self.connection2, self.ffn,
+                            self.post_norm2) if p is not None]
 
     def shift_need(self):
         """What the block's token shift keeps per request (None without one)."""
@@ -143,6 +154,10 @@ class Block(Part):
         if isinstance(delta, NormedSum) and (self.arrangement != "sandwich" or not getattr(self.norm1, "takes_normed_sum", False)):
             delta.settle(resid, self.rt.ops)
             delta = None
+        if (isinstance(delta, StreamUpdate) or resid.dim() == 3) and self.arrangement != "streams":
+            raise ValueError("a block of another arrangement cannot follow one that keeps several copies of the stream")
+        if self.arrangement == "streams":
+            return self._forward_streams(resid, delta, batch, cache, write_cache)
         if self.arrangement == "sandwich":
             return self._forward_sandwich(resid, delta, batch, cache, write_cache)
         if self.residual_scale is not None:
@@ -192,6 +207,17 @@ class Block(Part):
             return resid, left
         n2 = self.norm2.add_forward(resid, left)
         return resid, self._left_to_add(self.post_norm2, self.ffn.forward(n2, batch), resid)
+
+    def _forward_streams(self, resid, delta, batch, cache, write_cache):
+        """Several copies of the stream; the update that a sub-layer makes is left to the next reader."""
+        if delta is not None and not isinstance(delta, StreamUpdate):
+            raise ValueError("a block that keeps several copies of the stream takes the embedding's rows or such a block's update")
+        n1, resid = self.connection1.enter(resid, delta, self.norm1)
+        left = self.connection1.leave(self.mixer.forward(n1, batch, cache, write_cache))
+        if self.ffn is None:
+            return resid, left
+        n2, resid = self.connection2.enter(resid, left, self.norm2)
+        return resid, self.connection2.leave(self.ffn.forward(n2, batch))
 
     def _left_to_add(self, norm, y, resid):
         """norm(y) as something the next norm adds in its own pass, where both sides can; else it is added here."""

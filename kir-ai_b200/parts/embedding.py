@@ -1,4 +1,4 @@
-"""Token embedding (row gather; optionally times a constant and plus a sinusoidal position vector) and the output head.
+"""Token embedding (row gather; optionally times a constant and plus a sinusoidal or a learned position vector) and the output head.
 
 crates/llm-backend/src/core/qwen/ops/embedding.rs:26-36 (gather, error for an id outside
 the vocabulary) and crates/llm-backend/src/core/qwen/ops/lm_head.rs:68-86 of the
@@ -34,23 +34,30 @@ def sinusoid_frequencies(width: int, base: float) -> torch.Tensor:
 
 class Embedding(Part):
     """``scale`` multiplies the gathered rows; ``sinusoid_base`` b adds to the token at position p the vector whose
-    column 2i is sin(p b^(-2i/H)) and whose column 2i + 1 is the cosine of the same angle (angles in 32-bit).  With
-    neither, the rows are gathered as they are."""
+    column 2i is sin(p b^(-2i/H)) and whose column 2i + 1 is the cosine of the same angle (angles in 32-bit);
+    ``position_table`` = (tensor name, rows) adds the stored table's row of the token's position, unscaled.  With none of
+    them, the rows are gathered as they are."""
 
     capture_safe = True
     kernels_only = True
 
     def __init__(self, weight_name: str, vocab_size: int, hidden_size: int, *, scale: float = 1.0,
-                 sinusoid_base: Optional[float] = None):
+                 sinusoid_base: Optional[float] = None, position_table: Optional[tuple] = None):
         self.weight_name, self.vocab_size, self.hidden_size = weight_name, vocab_size, hidden_size
         self.scale, self.sinusoid_base = float(scale), sinusoid_base
-        self.uses_positions = sinusoid_base is not None
-        self.plain = self.scale == 1.0 and sinusoid_base is None
+        self.position_table_spec = position_table
+        self.uses_positions = sinusoid_base is not None or position_table is not None
+        self.plain = self.scale == 1.0 and not self.uses_positions
+        self.position_table: Optional[torch.Tensor] = None
         self.frequencies: Optional[torch.Tensor] = None
         self.table: Optional[torch.Tensor] = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
-        return {self.weight_name: WeightSpec((self.vocab_size, self.hidden_size), "embedding")}
+        specs = {self.weight_name: WeightSpec((self.vocab_size, self.hidden_size), "embedding")}
+        if self.position_table_spec is not None:
+            name, rows = self.position_table_spec
+            specs[name] = WeightSpec((rows, self.hidden_size), "embedding")
+        return specs
 
     def load(self, weights, rt: Runtime) -> None:
         self.rt = rt
@@ -60,12 +67,15 @@ class Embedding(Part):
         self.table = weights.on_device(self.weight_name, rt.dtype)
         if self.sinusoid_base is not None:
             self.frequencies = sinusoid_frequencies(self.hidden_size, self.sinusoid_base).to(rt.device)
+        if self.position_table_spec is not None:
+            self.position_table = weights.on_device(self.position_table_spec[0], rt.dtype)
 
     def forward(self, token_ids: torch.Tensor, positions: Optional[torch.Tensor] = None) -> torch.Tensor:
         """The 32-bit residual stream [T, H] that the blocks add into."""
         if self.plain:
             return self.rt.ops.embedding(self.table, token_ids)
-        stream, _ = self.rt.ops.embedding_scaled(self.table, token_ids, self.scale, positions, self.frequencies)
+        stream, _ = self.rt.ops.embedding_scaled(self.table, token_ids, self.scale, positions, self.frequencies,
+                                                position_table=self.position_table)
         return stream
 
     def forward_with_copy(self, token_ids: torch.Tensor, positions: Optional[torch.Tensor] = None):
@@ -74,7 +84,8 @@ class Embedding(Part):
         if self.plain:
             return self.forward(token_ids), None
         return self.rt.ops.embedding_scaled(self.table, token_ids, self.scale, positions, self.frequencies,
-                                            copy_dtype=None if self.rt.dtype == torch.float32 else self.rt.dtype)
+                                            copy_dtype=None if self.rt.dtype == torch.float32 else self.rt.dtype,
+                                            position_table=self.position_table)
 
 
 class OutputHead(Part):

@@ -11,7 +11,7 @@ from typing import Dict, Optional
 
 import torch
 
-from .base import FusedNormSpec, Norm, NormedSum, Runtime, ScaledSum, WeightSpec
+from .base import FusedNormSpec, Norm, NormedSum, Runtime, ScaledSum, StreamUpdate, WeightSpec
 
 
 class RMSNorm(Norm):
@@ -52,6 +52,13 @@ class RMSNorm(Norm):
             y = y.float()
         return self.rt.ops.norm_add(resid, y, self.weight, self.eps, None if self.rt.dtype == torch.float32 else self.rt.dtype)
 
+    takes_streams = True  # forward_streams, and add_forward_rows with a ``StreamUpdate`` (base.py)
+
+    def forward_streams(self, streams: torch.Tensor, copies: int, left, read: Optional[torch.Tensor]):
+        """(the normed rows of sum_t read[t] copy t after the update ``left``, the streams after it)."""
+        return self.rt.ops.streams_norm(streams, copies, left.terms() if left is not None else None, read, self.weight, self.eps,
+                                        self.rt.dtype)
+
     def fused_spec(self) -> Optional[FusedNormSpec]:
         # the tensor-core products read and write rows in 16-byte units; KIRAI_FUSE_NORMS=0 keeps every norm a
         # kernel of its own (for comparing the two paths)
@@ -60,7 +67,11 @@ class RMSNorm(Norm):
         return FusedNormSpec(self.weight, self.eps, self.width)
 
     def add_forward_rows(self, resid: torch.Tensor, delta: Optional[torch.Tensor], rows: torch.Tensor) -> torch.Tensor:
-        """The norm of ``resid[rows] + delta[rows]`` only; the stream is left untouched."""
+        """The norm of ``resid[rows] + delta[rows]`` only; the stream is left untouched.  With a ``StreamUpdate``: of the sum
+        of the copies after it."""
+        if isinstance(delta, StreamUpdate):
+            return self.rt.ops.streams_norm(resid, delta.mix.shape[0], delta.terms(), None, self.weight, self.eps, self.rt.dtype,
+                                            row_index=rows)[0]
         if isinstance(delta, NormedSum):
             return self.rt.ops.norm_add_norm(resid, delta.rows, delta.weight, delta.eps, self.weight, self.eps, self.rt.dtype,
                                              row_index=rows)

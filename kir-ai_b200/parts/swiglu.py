@@ -1,5 +1,6 @@
 """Dense gated feed-forward: down(act(gate x) * (up x)); act is silu(x) = x / (1 + e^-x) (SwiGLU) or, as
-``GatedMLP(activation="gelu_tanh")``, 0.5 x (1 + tanh(sqrt(2 / pi) (x + 0.044715 x^3))).
+``GatedMLP(activation="gelu_tanh")``, 0.5 x (1 + tanh(sqrt(2 / pi) (x + 0.044715 x^3))).  ``GatedMLP(activation="clamped",
+limit=L, slope=s)``: with g = min(gate x, L) and u = clamp(up x, -L, L), down(g sigmoid(s g) (u + 1)).
 
 crates/llm-backend/src/core/qwen/ops/moe.rs:31-88 and
 crates/llm-backend/src/core/math.rs:196-225 of the reference.  No biases.
@@ -19,6 +20,7 @@ class SwiGLU(FeedForward):
     kernels_only = True
 
     activation = "silu"
+    limit, slope = 0.0, 1.0  # of the clamped form
 
     def __init__(self, prefix: str, hidden_size: int, intermediate_size: int, names: Optional[Dict[str, str]] = None,
                  out_dtype: Optional[torch.dtype] = None):
@@ -62,22 +64,26 @@ class SwiGLU(FeedForward):
         """silu(gate x) * (up x): [T, I]."""
         ops = self.rt.ops
         if isinstance(x, UnscaledNorm):
-            return ops.linear_tcgen05(x.rows, self.fused_weight, swiglu=True, row_scale=x.row_scale(), gate_act=self.activation)
+            return ops.linear_tcgen05(x.rows, self.fused_weight, swiglu=True, row_scale=x.row_scale(), gate_act=self.activation,
+                                      gate_limit=self.limit, gate_slope=self.slope)
         if self.fused_weight is not None and ops.tcgen05_takes(x):
-            return ops.linear_tcgen05(x, self.fused_weight, swiglu=True, gate_act=self.activation)
+            return ops.linear_tcgen05(x, self.fused_weight, swiglu=True, gate_act=self.activation, gate_limit=self.limit, gate_slope=self.slope)
         if self.fused_weight is not None:
             raise ValueError("SwiGLU input is not laid out for the tensor-core kernel (rows must be 16-byte aligned)")
         if self.activation != "silu":
-            return ops.gated_activation(self.gate_up.forward(x), self.activation)
+            return ops.gated_activation(self.gate_up.forward(x), self.activation, self.limit, self.slope)
         return ops.swiglu(self.gate_up.forward(x))
 
 
 class GatedMLP(SwiGLU):
-    """The same feed-forward with the activation as an argument (``silu`` or ``gelu_tanh``)."""
+    """The same feed-forward with the activation as an argument (``silu``, ``gelu_tanh``, or ``clamped`` with its ``limit`` and ``slope``)."""
 
     def __init__(self, prefix: str, hidden_size: int, intermediate_size: int, activation: str = "silu",
-                 names: Optional[Dict[str, str]] = None, out_dtype: Optional[torch.dtype] = None):
-        if activation not in ("silu", "gelu_tanh"):
-            raise ValueError(f"unknown activation {activation!r}; known: silu, gelu_tanh")
+                 names: Optional[Dict[str, str]] = None, out_dtype: Optional[torch.dtype] = None, limit: float = 0.0, slope: float = 1.0):
+        if activation not in ("silu", "gelu_tanh", "clamped"):
+            raise ValueError(f"unknown activation {activation!r}; known: silu, gelu_tanh, clamped")
+        if (activation == "clamped") != (limit > 0.0):
+            raise ValueError("the clamped activation, and it alone, has a positive limit")
+        self.limit, self.slope = float(limit), float(slope)
         super().__init__(prefix, hidden_size, intermediate_size, names, out_dtype)
         self.activation = activation

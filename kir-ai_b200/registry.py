@@ -80,6 +80,10 @@ def _register_builtin() -> None:
     from .models.bikilix import build_bikilix_plan
 
     register_architecture(BikilixConfig.architecture, BikilixConfig, build_bikilix_plan, replace=True)
+    from .config.fosavik import FosavikConfig
+    from .models.fosavik import build_fosavik_plan
+
+    register_architecture(FosavikConfig.architecture, FosavikConfig, build_fosavik_plan, replace=True)
 
 
 _register_builtin()

@@ -2,7 +2,8 @@
 
 ``random_tensors`` fills every tensor that a model's parts declare, by role:
 linear matrices and embeddings from N(0, std), norm weights from
-1 + N(0, norm_jitter) (jitter 0 gives ones), integer tables uniformly.
+1 + N(0, norm_jitter) (jitter 0 gives ones), mixing matrices from the identity
+plus the same jitter, integer tables uniformly.
 ``write_random_model`` writes a model folder (config.json, model.safetensors).
 Tensors are generated one by one from a generator seeded with (seed, name), so
 a tensor's values do not depend on which other tensors exist or on the device
@@ -42,6 +43,8 @@ def random_tensors(specs: Mapping[str, WeightSpec], seed: int, *, std: float = 0
         values = torch.randn(spec.shape, generator=generator, device=device, dtype=torch.float32)
         if spec.role == "norm":
             values = 1.0 + norm_jitter * values
+        elif spec.role == "identity":
+            values = torch.eye(spec.shape[0], device=device) + norm_jitter * values
         else:
             values = std * values
         tensors[name] = values.to(dtype)
