@@ -331,8 +331,35 @@ def bikilix_config(size: dict, layers: int, intermediate: int) -> dict:
             "loop": {"start": 0, "stop": layers, "times": 1}}
 
 
+FOSAVIK_STREAMS = 4
+FOSAVIK_BLOCK = 256                                # channels of one block of the linear recurrence's gates
+FOSAVIK_WINDOW = dict(size=1024, keep_first=4)
+
+
+def fosavik_config(size: dict, layers: int, intermediate: int) -> dict:
+    """A Fosavik config.json of one size: four copies of the stream; layers in the order two-map attention, state space,
+    side by side, two-map attention over the keys and values of the first of the four (and so on), each with a dense clamped
+    feed-forward as large as the dense model's, the state space with none; two-map attention with the size's heads, two maps
+    of half a head's columns over values of a whole one's; the state-space mixer as in the Figalix configuration; the
+    attention side with the size's heads under a window of 1,024 that keeps four first keys; the recurrence as wide as the
+    model, in blocks of 256 channels."""
+    width, heads, kv_heads, dim = size["width"], size["heads"], size["kv_heads"], size["dim"]
+    pair = {"heads": heads, "kv_heads": kv_heads, "dim": dim // 2, "vdim": dim, "scale": (dim // 2) ** -0.5, "diff": 0.5}
+    state = {"heads": 2 * width // FIGALIX_STATE["vdim"], "vdim": FIGALIX_STATE["vdim"], "state": FIGALIX_STATE["state"], "groups": 1,
+             "conv": FIGALIX_STATE["conv"], "norm_groups": 1}
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": dict(FOSAVIK_WINDOW)}
+    side = {"left": left, "right": {"width": width, "blocks": width // FOSAVIK_BLOCK, "conv": 4}, "left_scale": 0.7, "right_scale": 0.9}
+    mlp = {"kind": "dense", "ff": intermediate, "limit": 7.0}
+    out = []
+    for i in range(layers):
+        kind, mixer = [("attention", pair), ("mamba2", state), ("parallel", side), ("attention", dict(pair, kv_from=i - 3))][i % 4]
+        out.append({"type": kind, "mixer": dict(mixer), "mlp": None if kind == "mamba2" else dict(mlp)})
+    return {"architecture": "Fosavik", "width": width, "vocab": size["vocab"], "max_positions": 8192, "streams": FOSAVIK_STREAMS,
+            "norm": {"eps": 1e-6}, "layers": out}
+
+
 def design_configs(size: dict, layers: int):
-    """(Zoferax config.json, Qwen3 config.json, Silupel config.json) of one size: the same width, heads and layer count;
+    """(Zoferax config.json, Qwen3 config.json, Silupel config.json and so on) of one size: the same width, heads and layer count;
     the dense feed-forward is as large as the experts that one token uses (3 I H = 2 top ff H)."""
     mixer = {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": size["dim"], "vdim": size["vdim"], "scale": size["dim"] ** -0.5}
     mlp = {"kind": "moe", "expert": {"ff": size["ff"]}, "router": {"experts": size["experts"], "top": size["top"]}}
@@ -344,7 +371,8 @@ def design_configs(size: dict, layers: int):
                  head_dim=size["dim"], vocab_size=size["vocab"], max_position_embeddings=40960, rms_norm_eps=1e-6,
                  rope_theta=1000000.0, tie_word_embeddings=False)
     return {"zoferax": zoferax, "qwen3-dense": dense, "silupel": silupel_config(size, layers, intermediate),
-            "figalix": figalix_config(size, layers, intermediate), "bikilix": bikilix_config(size, layers, intermediate)}
+            "figalix": figalix_config(size, layers, intermediate), "bikilix": bikilix_config(size, layers, intermediate),
+            "fosavik": fosavik_config(size, layers, intermediate)}
 
 
 def _kernel_rows(summary: dict, tokens: int, context_pairs: float, cache_rows: float, size: dict, design: str, peaks,
@@ -355,7 +383,7 @@ def _kernel_rows(summary: dict, tokens: int, context_pairs: float, cache_rows: f
     import re
 
     width, heads, kvh, dk = size["width"], size["heads"], size["kv_heads"], size["dim"]
-    dv = size["vdim"] if design in ("zoferax", "silupel", "figalix", "bikilix") else dk
+    dv = size["vdim"] if design in ("zoferax", "silupel", "figalix", "bikilix") else dk  # (fosavik: values of the size's key width)
     visible = visible or (lambda mask: (context_pairs, cache_rows))
     routed = size["experts"] * size["ff"]
     rows = []
@@ -363,7 +391,12 @@ def _kernel_rows(summary: dict, tokens: int, context_pairs: float, cache_rows: f
         flops = bytes_ = simt = 0.0
         label = name
         match = re.search(r"m=(\d+) n=(\d+) k=(\d+) form=(\d+)", name)
-        if match and "grouped" in name and design == "bikilix" and int(match.group(2)) == BIKILIX_LATENT["vdim"] \
+        if match and "grouped" in name and design == "fosavik":
+            # the recurrence's gates: two square matrices a block of channels over 32-bit rows (computed over two bfloat16 parts)
+            flops = 2.0 * tokens * width * 2 * FOSAVIK_BLOCK * count
+            bytes_ = (tokens * width * (4.0 + 8.0) + 4.0 * width * FOSAVIK_BLOCK) * count
+            label += " (the gates' blocks as groups)"
+        elif match and "grouped" in name and design == "bikilix" and int(match.group(2)) == BIKILIX_LATENT["vdim"] \
                 and int(match.group(3)) == BIKILIX_LATENT["kv_rank"] + BIKILIX_LATENT["rot_dim"]:
             # the heads' value matrices as groups over rows laid out head by head: the design's work is kv_rank columns a head
             h_, k_, n_ = BIKILIX_LATENT["heads"], BIKILIX_LATENT["kv_rank"], BIKILIX_LATENT["vdim"]
@@ -392,6 +425,8 @@ def _kernel_rows(summary: dict, tokens: int, context_pairs: float, cache_rows: f
             pairs, rows_read = visible(a_mask)
             shared = 1.0 if (design in ("silupel", "bikilix") and a_kv == 1) else 2.0  # a latent row is key and value in one
             flops = 2.0 * a_heads * 2 * a_d * pairs * count
+            if design == "fosavik" and a_mask == 0:  # a map's own half of the key row, and the whole value row
+                flops *= 0.75
             bytes_ = (2.0 * a_kv * shared * a_d * rows_read + 2.0 * tokens * a_heads * 2 * a_d) * count
         elif "attention" in name:
             flops = 2.0 * heads * (dk + dv) * context_pairs * count
@@ -399,6 +434,9 @@ def _kernel_rows(summary: dict, tokens: int, context_pairs: float, cache_rows: f
         elif "head_major" in name or "head_gate_rows" in name:
             bytes_ = tokens * BIKILIX_LATENT["heads"] * (4.0 * (BIKILIX_LATENT["kv_rank"] + BIKILIX_LATENT["rot_dim"]) if "major" in name
                                                           else 10.0 * BIKILIX_LATENT["vdim"]) * count
+        elif "head_linear_gate" in name and design == "fosavik":
+            # the gates' products of few tokens: their matrices once
+            bytes_ = (4.0 * width * FOSAVIK_BLOCK + tokens * width * 12.0) * count
         elif "head_linear_gate" in name:
             # a product per head between the attention over the shared latent and the output projection, and the gate
             t_, h_, k_, n_ = (int(v) for v in re.search(r"t=(\d+) heads=(\d+) k=(\d+) n=(\d+)", name).groups())
@@ -434,8 +472,22 @@ def _kernel_rows(summary: dict, tokens: int, context_pairs: float, cache_rows: f
                 cols = (width // 256) * (2 * FIGALIX_MEMORY["dim"] + 2 * FIGALIX_MEMORY["vdim"] + 2)
             simt = tokens * s_heads * (64.0 * (s_d + s_dv) + 4.0 * s_d * s_dv) * count
             bytes_ = (4.0 * tokens * cols + 8.0 * s_heads * s_d * s_dv * requests) * count
-        elif "conv_silu" in name:
-            bytes_ = tokens * (2 * width + 2 * FIGALIX_STATE["state"]) * 8.0 * count
+        elif "conv_rows" in name:
+            channels = int(re.search(r"c=(\d+)", name).group(1))
+            # (the linear recurrence's rows leave a second time, as two bfloat16 numbers each, for its gates' product)
+            bytes_ = tokens * channels * (8.0 + (4.0 if design == "fosavik" and channels == width and tokens >= 256 else 0.0)) * count
+        elif "streams_norm" in name:
+            # copies read and written in 32-bit, the sub-layer's output read, the normed rows written
+            first, update = "first" in name, "update" in name
+            values = (1 if first else FOSAVIK_STREAMS) * 4.0 + ((FOSAVIK_STREAMS + 1) * 4.0 if update and "rows" not in name else 0.0) + 2.0
+            bytes_ = (1 if "rows" in name else tokens) * width * values * count
+        elif "map_difference" in name:
+            bytes_ = tokens * heads * dk * 6.0 * count
+        elif "real_gated_step" in name:
+            # the gates' matrices once, a request's state and kept rows read and written
+            bytes_ = (4.0 * width * FOSAVIK_BLOCK + requests * width * (8.0 * 4 + 10.0)) * count
+        elif "real_gated_scan" in name:
+            bytes_ = (tokens * width * 18.0 + requests * width * 8.0) * count
         elif "gated_group_norm" in name:
             bytes_ = tokens * 2 * width * 10.0 * count
         elif "rms_pair_mean" in name:
@@ -624,7 +676,7 @@ def main() -> int:
                              "equal layer sizes (--sizes), with every step's time by kernel; a line of its own.")
     parser.add_argument("--sizes", default="2k,4k", help="layer sizes of --workload designs: " + ", ".join(DESIGN_SIZES))
     parser.add_argument("--designs", default="zoferax,qwen3-dense",
-                        help="which designs --workload designs measures, comma separated: zoferax, silupel, figalix, bikilix, qwen3-dense")
+                        help="which designs --workload designs measures, comma separated: zoferax, silupel, figalix, bikilix, fosavik, qwen3-dense")
     args = parser.parse_args()
 
     if args.impl == "reference":

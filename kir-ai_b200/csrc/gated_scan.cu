@@ -5,6 +5,7 @@
 //     taps - 1 rows more a run); the last taps - 1 rows that entered are state of the request.  For a product on the
 //     tensor cores that must not round its input to 16 bits the rows can leave a second time as two bfloat16 numbers
 //     each, high + low (16 bits of the value's 24), block by block of channels;
+//   * the whole of such a recurrence (convolution, gates, state, branch) for a step of single tokens as one kernel;
 //   * S_t = a_t S_(t-1) + b_t per channel, both terms from the current token alone: a block owns a few channels of one
 //     request and goes through the request's tokens in windows.  In a window every thread takes a run of TOKENS tokens of
 //     one channel: its terms stay in registers while the runs' (product of a, end state from zero) meet in shared memory,
@@ -168,6 +169,7 @@ struct RealGatedForm {
     static constexpr bool FAST = is_rounded<O>::value;
     struct Channel { float rb, ib, bb, rate; long gate_at; int c; };
     struct Row { float r, i, u, branch; };
+    using Kept = float;  // what the store of a token needs of its row
 
     __device__ __forceinline__ Channel channel(int c) const {
         const int b = c / block;
@@ -195,8 +197,9 @@ struct RealGatedForm {
             b = sqrtf(left) * (sf_sigmoid(row.i + ch.ib) * row.u);
         }
     }
-    __device__ __forceinline__ void store(const Channel& ch, const Row& row, long token, float s) const {
-        const float z = row.branch + ch.bb;
+    __device__ __forceinline__ Kept keep(const Row& row) const { return row.branch; }
+    __device__ __forceinline__ void store(const Channel& ch, Kept branch, long token, float s) const {
+        const float z = branch + ch.bb;
         // 0.5 z (1 + tanh(y)) = z sigmoid(2 y)
         const float gate = FAST ? __fdividef(z, 1.0f + __expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z))) : sf_gelu_tanh(z);
         out[token * out_stride + ch.c] = from_f32<O>(factor * (s * gate));
@@ -224,12 +227,12 @@ gated_scan_kernel(Form form, float* __restrict__ state, long state_len, long sta
     pdl_wait();
     float carry = live ? *kept : 0.0f;
     int turn = 0;
+    typename Form::Row row[TOKENS];
+#pragma unroll
+    for (int i = 0; i < TOKENS; ++i)
+        if (live && run * TOKENS + i < count) row[i] = form.load(ch, first + run * TOKENS + i);
     for (int w0 = 0; w0 < count; w0 += runs * TOKENS, turn ^= 1) {
         const int t0 = w0 + run * TOKENS;
-        typename Form::Row row[TOKENS];
-#pragma unroll
-        for (int i = 0; i < TOKENS; ++i)
-            if (live && t0 + i < count) row[i] = form.load(ch, first + t0 + i);
         float a[TOKENS], b[TOKENS];
         float prod = 1.0f, end = 0.0f;
 #pragma unroll
@@ -239,6 +242,14 @@ gated_scan_kernel(Form form, float* __restrict__ state, long state_len, long sta
             prod *= a[i];
             end = fmaf(a[i], end, b[i]);
         }
+        // the next window's rows are asked for here, ahead of the meeting and of this window's stores
+        typename Form::Kept held[TOKENS];
+#pragma unroll
+        for (int i = 0; i < TOKENS; ++i) held[i] = form.keep(row[i]);
+        const int next = t0 + runs * TOKENS;
+#pragma unroll
+        for (int i = 0; i < TOKENS; ++i)
+            if (live && next + i < count) row[i] = form.load(ch, first + next + i);
         float s = carry;
         if (runs > 1) {
             float2* here = ends + (size_t)turn * blockDim.x;
@@ -255,7 +266,7 @@ gated_scan_kernel(Form form, float* __restrict__ state, long state_len, long sta
 #pragma unroll
         for (int i = 0; i < TOKENS; ++i) {
             s = fmaf(a[i], s, b[i]);
-            if (live && t0 + i < count) form.store(ch, row[i], first + t0 + i, s);
+            if (live && t0 + i < count) form.store(ch, held[i], first + t0 + i, s);
         }
     }
     // (every thread of the channel read the old state ahead of its first barrier, or is the only one)
@@ -297,7 +308,190 @@ int real_gated_launch(const float* u, const float* gates, long gate_token, long 
     return gated_scan_launch(form, state, state_len, state_off, query_start, slots, requests, max_query_len, channels, num_slots, stream);
 }
 
+// ------------------------------------------------------------------ a step of single tokens
+// Convolution, the gates' products, the recurrence and the gelu branch for a step in which every request brings one token
+// (row r is request r's).  A cluster of CTAs takes a block of channels; every CTA makes the block's u for STEP_ROWS requests
+// at a time in its own shared memory, multiplies it with the rows of its share of the block's two gate matrices (a warp
+// per channel, 32-bit multiply-adds, the lanes' partial sums of all requests folded together), and finishes its channels.
+// The kept rows of the convolution are read by the whole cluster: they move on after the cluster has met.
+#define STEP_ROWS 8
+
+template <typename W>
+__device__ __forceinline__ float4 weights4(const W* p);
+template <>
+__device__ __forceinline__ float4 weights4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <>
+__device__ __forceinline__ float4 weights4<bf16>(const bf16* p) {
+    const uint2 q = *reinterpret_cast<const uint2*>(p);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+    return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+
+struct StepArgs {
+    const float* rows;  // [R, >= 2 width], row stride: the branch's columns, then the convolution's input
+    long row_stride;
+    const float *taps_w, *in_bias, *bias;
+    const void* gates;  // [blocks, 2 block, block]
+    const float *r_bias, *i_bias, *branch_bias, *rate;
+    float factor;
+    float* state;
+    long state_len, conv_off, state_off;
+    const int* slots;
+    long out_stride;
+    int requests, width, block, taps, num_slots;
+};
+
+template <typename O, typename W, bool VEC>
+__global__ void __launch_bounds__(256) real_gated_step_kernel(StepArgs a, O* __restrict__ out) {
+    pdl_launch_dependents();
+    extern __shared__ float step_smem[];
+    const int d = a.block, cuts = gridDim.x, b = blockIdx.y;
+    const int per = (d + cuts - 1) / cuts;
+    const int lo = min(d, (int)blockIdx.x * per), hi = min(d, lo + per);
+    float* u_s = step_smem;                    // [STEP_ROWS][d]
+    float* gate_s = step_smem + STEP_ROWS * d;  // [2][STEP_ROWS][per]
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    const W* gates = reinterpret_cast<const W*>(a.gates) + (size_t)b * 2 * d * d;
+    // this CTA's rows of the two matrices, asked into L2 while the kernel before still runs
+    for (int gate = 0; gate < 2; ++gate) {
+        const char* from = reinterpret_cast<const char*>(gates + ((size_t)gate * d + lo) * d);
+        const size_t bytes = (size_t)(hi - lo) * d * sizeof(W);
+        for (size_t at = threadIdx.x * 128u; at < bytes; at += blockDim.x * 128u) asm volatile("prefetch.global.L2 [%0];" ::"l"(from + at));
+    }
+    pdl_wait();
+    const int taps = a.taps, width = a.width;
+    for (int r0 = 0; r0 < a.requests; r0 += STEP_ROWS) {
+        const int count = min(STEP_ROWS, a.requests - r0);
+        if (r0) __syncthreads();
+        for (int at = threadIdx.x; at < STEP_ROWS * d; at += blockDim.x) {
+            const int r = at / d, c = b * d + (at - r * d);
+            float acc = 0.0f;
+            if (r < count) {
+                const int slot = a.slots[r0 + r];
+                if (slot >= 0 && slot < a.num_slots) {
+                    const float* kept = a.state + (long)slot * a.state_len + a.conv_off + c;
+                    acc = a.bias[c];
+                    for (int j = 0; j + 1 < taps; ++j) acc = fmaf(a.taps_w[(long)c * taps + j], kept[(long)j * width], acc);
+                    acc = fmaf(a.taps_w[(long)c * taps + taps - 1], a.rows[(r0 + r) * a.row_stride + width + c] + a.in_bias[c], acc);
+                }
+            }
+            u_s[at] = acc;
+        }
+        __syncthreads();
+        for (int j = lo + warp; j < hi; j += warps) {
+            const W* row_r = gates + (size_t)j * d;
+            const W* row_i = gates + (size_t)(d + j) * d;
+            float sum[2 * STEP_ROWS];  // the requests' r sums, then their i sums
+#pragma unroll
+            for (int r = 0; r < 2 * STEP_ROWS; ++r) sum[r] = 0.0f;
+            if (VEC) {
+                for (int k = lane * 4; k < d; k += 128) {
+                    const float4 wr = weights4<W>(row_r + k), wi = weights4<W>(row_i + k);
+#pragma unroll
+                    for (int r = 0; r < STEP_ROWS; ++r) {
+                        const float4 u = *reinterpret_cast<const float4*>(u_s + r * d + k);
+                        sum[r] = fmaf(wr.x, u.x, fmaf(wr.y, u.y, fmaf(wr.z, u.z, fmaf(wr.w, u.w, sum[r]))));
+                        sum[STEP_ROWS + r] = fmaf(wi.x, u.x, fmaf(wi.y, u.y, fmaf(wi.z, u.z, fmaf(wi.w, u.w, sum[STEP_ROWS + r]))));
+                    }
+                }
+            } else {
+                for (int k = lane; k < d; k += 32) {
+                    const float wr = to_f32<W>(row_r[k]), wi = to_f32<W>(row_i[k]);
+#pragma unroll
+                    for (int r = 0; r < STEP_ROWS; ++r) {
+                        sum[r] = fmaf(wr, u_s[r * d + k], sum[r]);
+                        sum[STEP_ROWS + r] = fmaf(wi, u_s[r * d + k], sum[STEP_ROWS + r]);
+                    }
+                }
+            }
+            // sixteen sums over 32 lanes: halves change hands until a lane holds one sum, then the last two lanes add up
+#pragma unroll
+            for (int half = STEP_ROWS, lanes = 16; half >= 1; half >>= 1, lanes >>= 1) {
+                const bool upper = (lane & lanes) != 0;
+#pragma unroll
+                for (int r = 0; r < half; ++r) {
+                    const float give = upper ? sum[r] : sum[half + r];
+                    const float got = __shfl_xor_sync(0xffffffffu, give, lanes);
+                    sum[r] = (upper ? sum[half + r] : sum[r]) + got;
+                }
+            }
+            const float total = sum[0] + __shfl_xor_sync(0xffffffffu, sum[0], 1);
+            // lane bits 4, 3, 2, 1 say which sum it is, the highest first
+            const int which = lane >> 1;
+            if ((lane & 1) == 0) gate_s[which * per + (j - lo)] = total;
+        }
+        __syncthreads();
+        for (int at = threadIdx.x; at < count * (hi - lo); at += blockDim.x) {
+            const int r = at / (hi - lo), j = at - r * (hi - lo);
+            const int slot = a.slots[r0 + r];
+            if (slot < 0 || slot >= a.num_slots) continue;
+            const int c = b * d + lo + j;
+            const RealGatedForm<O> form{nullptr, nullptr, 0, 0, d, nullptr, 0, a.r_bias, a.i_bias, a.branch_bias, a.rate, a.factor, out, a.out_stride, width};
+            const typename RealGatedForm<O>::Channel ch = form.channel(c);
+            const typename RealGatedForm<O>::Row row{gate_s[r * per + j], gate_s[(STEP_ROWS + r) * per + j], u_s[r * d + lo + j],
+                                                     a.rows[(r0 + r) * a.row_stride + c]};
+            float* S = a.state + (long)slot * a.state_len + a.state_off + c;
+            float keep, take;
+            form.terms(ch, row, keep, take);
+            const float s = fmaf(keep, *S, take);
+            *S = s;
+            form.store(ch, form.keep(row), r0 + r, s);
+        }
+    }
+    // every CTA of the cluster has read the block's kept rows
+    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+    if (taps > 1) {
+        for (int at = threadIdx.x; at < a.requests * (hi - lo); at += blockDim.x) {
+            const int r = at / (hi - lo), c = b * d + lo + (at - r * (hi - lo));
+            const int slot = a.slots[r];
+            if (slot < 0 || slot >= a.num_slots) continue;
+            float* kept = a.state + (long)slot * a.state_len + a.conv_off + c;
+            for (int k = 0; k + 2 < taps; ++k) kept[(long)k * width] = kept[(long)(k + 1) * width];
+            kept[(long)(taps - 2) * width] = a.rows[r * a.row_stride + width + c] + a.in_bias[c];
+        }
+    }
+}
+
+template <typename O>
+int real_gated_step_launch(const StepArgs& a, int gates_bf16, void* out, cudaStream_t stream) {
+    if (a.requests <= 0) return 0;
+    if (a.width <= 0 || a.block <= 0 || a.width % a.block || a.taps < 1 || a.conv_off < 0 || a.state_off < 0 || a.out_stride < a.width ||
+        a.conv_off + (long)(a.taps - 1) * a.width > a.state_len || a.state_off + a.width > a.state_len)
+        return KIRAI_ERR_BAD_SIZE;
+    const int blocks = a.width / a.block;
+    if (blocks > 65535) return KIRAI_ERR_BAD_SIZE;
+    int cuts = 1;
+    while (cuts < 8 && blocks * cuts < 148 && a.block / (cuts * 2) >= 8) cuts *= 2;
+    const int per = (a.block + cuts - 1) / cuts;
+    const size_t smem = (size_t)STEP_ROWS * (a.block + 2 * per) * sizeof(float);
+    if (smem > 200 * 1024) return KIRAI_ERR_BAD_SIZE;
+    const bool vec = a.block % 4 == 0 && ((uintptr_t)a.gates & 15) == 0;
+    auto kernel = gates_bf16 ? (vec ? real_gated_step_kernel<O, bf16, true> : real_gated_step_kernel<O, bf16, false>)
+                             : (vec ? real_gated_step_kernel<O, float, true> : real_gated_step_kernel<O, float, false>);
+    if (smem > 48 * 1024) {
+        const cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (err != cudaSuccess) return (int)err;
+    }
+    return launch_pdl_clusters(kernel, dim3(cuts, blocks), dim3(256), smem, stream, dim3(cuts, 1, 1), a, (O*)out);
+}
+
 }  // namespace
+
+// A step of single tokens in one kernel (see real_gated_step_kernel): the kept rows at columns [conv_off, conv_off +
+// (taps - 1) width) of the request's slot, S at [state_off, state_off + width).
+#define KIRAI_REAL_GATED_STEP(NAME, O)                                                                                            \
+    KIRAI_EXPORT int NAME(const float* rows, long row_stride, const float* taps_w, const float* in_bias, const float* bias,       \
+                          const void* gates, int gates_bf16, const float* r_bias, const float* i_bias, const float* branch_bias, \
+                          const float* rate, float factor, float* state, long state_len, long conv_off, long state_off,          \
+                          const int* slots, void* out, long out_stride, int requests, int width, int block, int taps,            \
+                          int num_slots, cudaStream_t stream) {                                                                  \
+        const StepArgs a{rows, row_stride, taps_w, in_bias, bias, gates, r_bias, i_bias, branch_bias, rate, factor, state,       \
+                         state_len, conv_off, state_off, slots, out_stride, requests, width, block, taps, num_slots};            \
+        return real_gated_step_launch<O>(a, gates_bf16, out, stream);                                                            \
+    }
+KIRAI_REAL_GATED_STEP(kirai_real_gated_step_f32, float)
+KIRAI_REAL_GATED_STEP(kirai_real_gated_step_bf16, bf16)
+#undef KIRAI_REAL_GATED_STEP
 
 // out [T, channels] (float32) = (silu of) bias + sum_j taps_w[c, j] * (in[t - (taps - 1) + j, c] + in_bias[c]) per request,
 // kept rows before a request's first row of this step; then the kept rows move on.  pair (may be null): the same rows as

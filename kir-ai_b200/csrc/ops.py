@@ -784,6 +784,32 @@ def real_gated_scan(u: torch.Tensor, gates: torch.Tensor, block: int, branch: to
     return out
 
 
+def real_gated_step_takes(batch, block: int) -> bool:
+    """Whether ``real_gated_step`` takes this step: every request brings one token, and a block's rows fit shared memory."""
+    return batch.decode_only and batch.num_requests <= 128 and block <= 2048
+
+
+def real_gated_step(rows: torch.Tensor, width: int, block: int, taps: torch.Tensor, in_bias: torch.Tensor, bias: torch.Tensor,
+                    gates: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor, branch_bias: torch.Tensor, rate: torch.Tensor,
+                    state: torch.Tensor, conv_offset: int, state_offset: int, batch, out: torch.Tensor, factor: float = 1.0) -> torch.Tensor:
+    """``conv_rows``, ``block_product`` and ``real_gated_scan`` in one kernel for a step of single tokens: ``rows`` [R, >= 2
+    width] (float32: the branch's columns, then the convolution's input), ``gates`` [blocks, 2 block, block] (bfloat16 or
+    float32; 32-bit multiply-adds either way); everything else as there."""
+    _need_cuda(rows, taps, in_bias, bias, gates, r_bias, i_bias, branch_bias, rate, state, out)
+    assert rows.dtype == torch.float32 and rows.dim() == 2 and rows.stride(1) == 1 and rows.shape[1] >= 2 * width
+    for t in (in_bias, bias, r_bias, i_bias, branch_bias, rate):
+        assert t.dtype == torch.float32 and t.numel() == width and t.is_contiguous()
+    assert taps.dtype == torch.float32 and taps.dim() == 2 and taps.shape[0] == width and taps.is_contiguous()
+    assert gates.shape == (width // block, 2 * block, block) and gates.is_contiguous() and gates.dtype in (torch.float32, torch.bfloat16)
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous()
+    assert out.shape == (rows.shape[0], width) and out.stride(1) == 1 and rows.shape[0] == batch.num_requests
+    _call(f"kirai_real_gated_step_{_suffix(out.dtype)}", _ptr(rows), _l(rows.stride(0)), _ptr(taps), _ptr(in_bias), _ptr(bias), _ptr(gates),
+          _i(int(gates.dtype == torch.bfloat16)), _ptr(r_bias), _ptr(i_bias), _ptr(branch_bias), _ptr(rate), _f(factor), _ptr(state),
+          _l(state.shape[1]), _l(conv_offset), _l(state_offset), _ptr(batch.slots), _ptr(out), _l(out.stride(0)), _i(rows.shape[0]),
+          _i(width), _i(block), _i(taps.shape[1]), _i(state.shape[0]), _stream())
+    return out
+
+
 def streams_norm(streams: torch.Tensor, copies: int, update: Optional[tuple], read: Optional[torch.Tensor], weight: Optional[torch.Tensor],
                  eps: float, out_dtype: torch.dtype, row_index: Optional[torch.Tensor] = None):
     """A stream of ``copies`` copies read through a norm, after the update that the sub-layer before left: ``streams`` is

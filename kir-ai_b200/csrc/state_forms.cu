@@ -144,12 +144,80 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, long y_stri
     }
 }
 
+// The same with 16-byte loads, a block of up to 1,024 threads per (row, group), the gated values in registers between the
+// statistics and the output (group width a multiple of 4, at most 4 * VEC * blockDim values; aligned rows).
+template <typename O, int VEC>
+__global__ void __launch_bounds__(1024) gated_group_norm_vec_kernel(const float* __restrict__ y, long y_stride, const float* __restrict__ gate,
+                                                                    long g_stride, const float* __restrict__ weight, float eps,
+                                                                    O* __restrict__ out, int groups, int group_width, int mode) {
+    __shared__ float scratch[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const long row = blockIdx.x / groups;
+    const int c0 = (int)(blockIdx.x - row * groups) * group_width;
+    const float* py = y + row * y_stride + c0;
+    const float* pg = gate + row * g_stride + c0;
+    float4 v[VEC], g[VEC];
+    float sum = 0.0f;
+#pragma unroll
+    for (int n = 0; n < VEC; ++n) {
+        const int c = (threadIdx.x + n * blockDim.x) * 4;
+        if (c >= group_width) break;
+        v[n] = *reinterpret_cast<const float4*>(py + c);
+        g[n] = *reinterpret_cast<const float4*>(pg + c);
+    }
+#pragma unroll
+    for (int n = 0; n < VEC; ++n) {
+        const int c = (threadIdx.x + n * blockDim.x) * 4;
+        if (c >= group_width) break;
+        if (mode == 0) v[n].x *= sf_silu(g[n].x), v[n].y *= sf_silu(g[n].y), v[n].z *= sf_silu(g[n].z), v[n].w *= sf_silu(g[n].w);
+        sum += (v[n].x * v[n].x + v[n].y * v[n].y) + (v[n].z * v[n].z + v[n].w * v[n].w);
+        if (mode != 0) v[n].x *= sf_sigmoid(g[n].x), v[n].y *= sf_sigmoid(g[n].y), v[n].z *= sf_sigmoid(g[n].z), v[n].w *= sf_sigmoid(g[n].w);
+    }
+    sum = block_sum(sum, scratch);
+    const float r = rsqrtf(sum / (float)group_width + eps);
+    O* po = out + row * (long)groups * group_width + c0;
+#pragma unroll
+    for (int n = 0; n < VEC; ++n) {
+        const int c = (threadIdx.x + n * blockDim.x) * 4;
+        if (c >= group_width) break;
+        const float4 w = *reinterpret_cast<const float4*>(weight + c0 + c);
+        const float a = v[n].x * r * w.x, b = v[n].y * r * w.y, d = v[n].z * r * w.z, e = v[n].w * r * w.w;
+        if (sizeof(O) == 4) {
+            *reinterpret_cast<float4*>(po + c) = make_float4(a, b, d, e);
+        } else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(d, e);
+            uint2 packed;
+            packed.x = *reinterpret_cast<const uint32_t*>(&lo);
+            packed.y = *reinterpret_cast<const uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>(po + c) = packed;
+        }
+    }
+}
+
 template <typename O>
 static int gated_group_norm_launch(const float* y, long y_stride, const float* gate, long g_stride, const float* weight, float eps,
                                    void* out, int rows, int groups, int group_width, int mode, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (groups <= 0 || group_width <= 0 || mode < 0 || mode > 1) return KIRAI_ERR_BAD_SIZE;
     const long units = (long)rows * groups;
+    const bool vec = group_width % 4 == 0 && group_width >= 512 && group_width <= 4 * 4 * 1024 && y_stride % 4 == 0 && g_stride % 4 == 0 &&
+                     (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+    if (vec) {
+        // many units: four pieces a thread; few: one or two, so that a row's loads are all in flight at once
+        const int quads = group_width / 4;
+        const int per = units > 296 ? 4 : 1;
+        int threads = ((quads + per - 1) / per + 31) / 32 * 32;
+        if (threads > 1024) threads = 1024;
+        if (quads <= threads)
+            return launch_pdl(gated_group_norm_vec_kernel<O, 1>, dim3((unsigned)units), dim3(threads), 0, stream, 1u, y, y_stride, gate, g_stride,
+                              weight, eps, (O*)out, groups, group_width, mode);
+        if (quads <= 2 * threads)
+            return launch_pdl(gated_group_norm_vec_kernel<O, 2>, dim3((unsigned)units), dim3(threads), 0, stream, 1u, y, y_stride, gate, g_stride,
+                              weight, eps, (O*)out, groups, group_width, mode);
+        return launch_pdl(gated_group_norm_vec_kernel<O, 4>, dim3((unsigned)units), dim3(threads), 0, stream, 1u, y, y_stride, gate, g_stride,
+                          weight, eps, (O*)out, groups, group_width, mode);
+    }
     if (group_width >= 512)
         return launch_pdl(gated_group_norm_kernel<O, 8>, dim3((unsigned)units), dim3(256), 0, stream, 1u, y, y_stride, gate, g_stride,
                           weight, eps, (O*)out, (long)rows, groups, group_width, mode);

@@ -44,7 +44,7 @@ __device__ __forceinline__ void fma_quad(float4& acc, float a, const float4& x) 
 // One block per produced row, 16-byte accesses; a thread owns the same columns of every copy, so the update in place
 // needs no barrier; u stays in registers between the statistics and the output.
 template <typename T, int S, int VEC>
-__global__ void streams_norm_vec_kernel(StreamArgs a, T* __restrict__ out) {
+__global__ void __launch_bounds__(VEC == 4 ? 512 : 1024) streams_norm_vec_kernel(StreamArgs a, T* __restrict__ out) {
     pdl_launch_dependents();
     __shared__ float scratch[32];
     // the coefficients are weights: read before the wait
@@ -63,16 +63,28 @@ __global__ void streams_norm_vec_kernel(StreamArgs a, T* __restrict__ out) {
     float* dst = a.dst ? a.dst + row * S * (size_t)a.width : nullptr;
     float4 u[VEC];
     float acc = 0.0f;
+    // (src and dst may be the same rows: every load of a pair of pieces stands ahead of its stores)
+    constexpr int AHEAD = VEC >= 2 ? 2 : 1;
 #pragma unroll
-    for (int n = 0; n < VEC; ++n) {
+    for (int n0 = 0; n0 < VEC; n0 += AHEAD) {
+    float4 old[AHEAD][S], new_y[AHEAD];
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) {
+        const int c = (threadIdx.x + (n0 + k) * blockDim.x) * 4;
+        if (c >= a.width) continue;
+#pragma unroll
+        for (int f = 0; f < S; ++f) old[k][f] = *reinterpret_cast<const float4*>(src + f * a.src_copy + c);
+        if (y) new_y[k] = *reinterpret_cast<const float4*>(y + c);
+    }
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) {
+        const int n = n0 + k;
         const int c = (threadIdx.x + n * blockDim.x) * 4;
         u[n] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if (c >= a.width) continue;
-        float4 x[S];
-#pragma unroll
-        for (int f = 0; f < S; ++f) x[f] = *reinterpret_cast<const float4*>(src + f * a.src_copy + c);
+        const float4 (&x)[S] = old[k];
         if (y) {
-            const float4 v = *reinterpret_cast<const float4*>(y + c);
+            const float4 v = new_y[k];
 #pragma unroll
             for (int t = 0; t < S; ++t) {
                 float4 now = make_float4(add[t] * v.x, add[t] * v.y, add[t] * v.z, add[t] * v.w);
@@ -86,6 +98,7 @@ __global__ void streams_norm_vec_kernel(StreamArgs a, T* __restrict__ out) {
             for (int f = 0; f < S; ++f) fma_quad(u[n], read[f], x[f]);
         }
         acc += (u[n].x * u[n].x + u[n].y * u[n].y) + (u[n].z * u[n].z + u[n].w * u[n].w);
+    }
     }
     float scale = 1.0f;
     if (a.weight) {
@@ -159,9 +172,18 @@ int streams_norm_launch(const StreamArgs& a, void* out, int rows, cudaStream_t s
     const bool aligned = a.width % 4 == 0 && a.src_token % 4 == 0 && a.src_copy % 4 == 0 &&
                          (((uintptr_t)a.src | (uintptr_t)a.dst | (uintptr_t)a.y | (uintptr_t)a.weight | (uintptr_t)out) & 15) == 0;
     if (aligned && a.copies <= 4 && a.width <= 4 * 4 * 512) {
-        const int threads = a.width <= 4 * 4 * 128 ? 128 : (a.width <= 4 * 4 * 256 ? 256 : 512);
+        // few rows: as many threads a row as it has pieces, so that all of it is asked for at once
+        const int quads = a.width / 4;
+        const bool few = rows <= 148;
+        const int threads = few ? (quads <= 1024 ? (quads + 31) / 32 * 32 : 1024)
+                                : (a.width <= 4 * 4 * 128 ? 128 : (a.width <= 4 * 4 * 256 ? 256 : 512));
+        const int vec = few ? (quads + threads - 1) / threads : 4;
 #define KIRAI_STREAMS(S)                                                                                                       \
     case S:                                                                                                                   \
+        if (vec == 1)                                                                                                         \
+            return launch_pdl(streams_norm_vec_kernel<T, S, 1>, dim3(rows), dim3(threads), 0, stream, 1u, a, (T*)out);        \
+        if (vec == 2)                                                                                                         \
+            return launch_pdl(streams_norm_vec_kernel<T, S, 2>, dim3(rows), dim3(threads), 0, stream, 1u, a, (T*)out);        \
         return launch_pdl(streams_norm_vec_kernel<T, S, 4>, dim3(rows), dim3(threads), 0, stream, 1u, a, (T*)out)
         switch (a.copies) {
             KIRAI_STREAMS(1);

@@ -12,7 +12,7 @@ What a request keeps between steps is one slot row in 32-bit: the convolution's 
 their bias), then S; both start at zero.  The stacked input product leaves 32-bit rows; convolution, gates, decays and the
 recurrence are 32-bit.  The gates' products run in 32-bit multiply-adds, or, for steps of many tokens in bfloat16, on the
 tensor cores with u as two bfloat16 numbers, high + low (``ops.block_product_pairs``), so that u is not rounded to 16 bits
-ahead of a gate either way.
+ahead of a gate either way.  A step of single tokens runs everything between the outer products as one kernel.
 """
 from __future__ import annotations
 
@@ -86,6 +86,8 @@ class GatedLinearRecurrence(Mixer):
         self.rate = (-self.decay * torch.nn.functional.softplus(lam, threshold=40.0)).to(torch.float32).contiguous()
         stacked = torch.cat([weights.stored(n[key]).to(device=rt.device) for key in ("r", "i")], dim=1)  # [blocks, 2 d, d]
         self.gates = stacked.to(torch.float32).contiguous()
+        # (what a step of single tokens reads: stored bfloat16 matrices as they are, which changes no product)
+        self.step_gates = stacked.contiguous() if stacked.dtype == torch.bfloat16 else self.gates
         self.gate_pairs = None
         if rt.dtype == torch.bfloat16 and d % 4 == 0 and stacked.dtype == torch.bfloat16:
             pairs = torch.cat([stacked, stacked], dim=2).reshape(self.blocks * 2 * d, 2 * d).contiguous()
@@ -95,6 +97,9 @@ class GatedLinearRecurrence(Mixer):
         """Everything between the products: ``rows`` [T, 2 width] (float32, what the input matrices made: y, then x) to
         ``out`` [T, width], what the output projection reads, times ``factor``."""
         ops, tokens = self.rt.ops, rows.shape[0]
+        if ops.real_gated_step_takes(batch, self.block):
+            return ops.real_gated_step(rows, self.width, self.block, self.conv, self.x_bias, self.conv_bias, self.step_gates, self.r_bias,
+                                       self.i_bias, self.y_bias, self.rate, cache.state, 0, self.conv_len, batch, out, factor)
         branch, x = rows[:, : self.width], rows[:, self.width : 2 * self.width]
         if self.gate_pairs is not None and tokens >= self.PAIRS_MIN_ROWS:
             u, pair = ops.conv_rows(x, self.conv, self.conv_bias, cache.state, 0, batch, in_bias=self.x_bias, pair_block=self.block,
