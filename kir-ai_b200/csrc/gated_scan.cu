@@ -32,7 +32,7 @@ struct ConvArgs {
     const float* taps_w;   // [channels, taps], the last column weighs the token itself
     const float* in_bias;  // [channels] or null: added to every row that enters (zeros lie before a sequence's start)
     const float* bias;     // [channels] or null
-    const float* state;    // [slots, state_len], kept rows [taps - 1, channels] from column conv_off, the newest last
+    float* state;          // [slots, state_len], kept rows [taps - 1, channels] from column conv_off, the newest last
     long state_len, conv_off;
     const int* request_of_token;
     const int* query_start;
@@ -41,6 +41,8 @@ struct ConvArgs {
     bf16* pair;    // null, or [channels / block, pair_tokens, 2 * block]: high parts, then low parts
     int block, pair_tokens;
     int tokens, channels, num_slots, silu;
+    int run;     // tokens a block walks, at most CONV_RUN
+    int single;  // every request brings one token: the thread that read a channel's kept rows moves them on itself
 };
 
 __device__ __forceinline__ void conv_store(const ConvArgs& a, long token, int c, float v) {
@@ -60,8 +62,8 @@ __global__ void conv_run_kernel(ConvArgs a) {
     pdl_launch_dependents();
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
     if (c >= a.channels) return;
-    const long t0 = (long)blockIdx.x * CONV_RUN;
-    const int count = (int)min((long)CONV_RUN, a.tokens - t0);
+    const long t0 = (long)blockIdx.x * a.run;
+    const int count = (int)min((long)a.run, a.tokens - t0);
     float w[TAPS];
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) w[j] = a.taps_w[(long)c * TAPS + j];
@@ -84,12 +86,16 @@ __global__ void conv_run_kernel(ConvArgs a) {
             const long first = a.query_start[current];
             const int local = (int)(t0 + i - first);
             const int slot = a.slots[current];
-            const float* kept = a.state + (long)slot * a.state_len + a.conv_off;
+            float* kept = a.state + (long)slot * a.state_len + a.conv_off;
             const bool held = slot >= 0 && slot < a.num_slots;
 #pragma unroll
             for (int j = 0; j < TAPS - 1; ++j) {
                 const int at = local - (TAPS - 1) + j;
                 past[j] = at >= 0 ? a.in[(first + at) * a.in_stride + c] + in_bias : (held ? kept[(long)(TAPS - 1 + at) * a.channels + c] : 0.0f);
+            }
+            if (a.single && held) {
+#pragma unroll
+                for (int j = 0; j < TAPS - 1; ++j) kept[(long)j * a.channels + c] = j + 1 < TAPS - 1 ? past[j + 1] : x[i];
             }
         }
         float acc = bias;
@@ -208,7 +214,7 @@ struct RealGatedForm {
 
 // Blocks (run of CH channels, request); threads: `runs` * CH.
 template <class Form, int CH, int TOKENS>
-__global__ void __launch_bounds__(512)
+__global__ void __launch_bounds__(256)
 gated_scan_kernel(Form form, float* __restrict__ state, long state_len, long state_off, const int* __restrict__ query_start,
                   const int* __restrict__ slots, int channels, int num_slots) {
     pdl_launch_dependents();
@@ -277,21 +283,18 @@ template <class Form>
 int gated_scan_launch(const Form& form, float* state, long state_len, long state_off, const int* query_start, const int* slots,
                       int requests, int max_query_len, int channels, int num_slots, cudaStream_t stream) {
     constexpr int TOKENS = 8;
-    // a warp's row is one line of 32 channels; where that leaves processors without a block, 16 channels
-    const bool narrow = (long)((channels + 31) / 32) * requests < 148;
-    const int ch = narrow ? 16 : 32;
+    // a warp's rows are runs of 32 channels (one line), or of 16 or 8 (whole sectors) where that brings two blocks to an SM
+    int ch = 32;
+    while (ch > 8 && (long)((channels + ch - 1) / ch) * requests < 256) ch >>= 1;
     int runs = (max_query_len + TOKENS - 1) / TOKENS;
-    const int most = 512 / ch, least = 32 / ch;
+    const int most = 256 / ch, least = 32 / ch;
     if (runs > most) runs = most;
     if (runs < least) runs = least;
     const int threads = ((runs * ch + 31) / 32) * 32;
     const size_t smem = 2 * (size_t)threads * sizeof(float2);
     const dim3 grid((channels + ch - 1) / ch, requests);
-    if (narrow)
-        return launch_pdl(gated_scan_kernel<Form, 16, TOKENS>, grid, dim3(threads), smem, stream, 1u, form, state, state_len, state_off,
-                          query_start, slots, channels, num_slots);
-    return launch_pdl(gated_scan_kernel<Form, 32, TOKENS>, grid, dim3(threads), smem, stream, 1u, form, state, state_len, state_off,
-                      query_start, slots, channels, num_slots);
+    auto kernel = ch == 32 ? gated_scan_kernel<Form, 32, TOKENS> : ch == 16 ? gated_scan_kernel<Form, 16, TOKENS> : gated_scan_kernel<Form, 8, TOKENS>;
+    return launch_pdl(kernel, grid, dim3(threads), smem, stream, 1u, form, state, state_len, state_off, query_start, slots, channels, num_slots);
 }
 
 template <typename O>
@@ -315,14 +318,15 @@ int real_gated_launch(const float* u, const float* gates, long gate_token, long 
 // per channel, 32-bit multiply-adds, the lanes' partial sums of all requests folded together), and finishes its channels.
 // The kept rows of the convolution are read by the whole cluster: they move on after the cluster has met.
 #define STEP_ROWS 8
+#define STEP_REQUESTS 128
 
 template <typename W>
 __device__ __forceinline__ float4 weights4(const W* p);
 template <>
-__device__ __forceinline__ float4 weights4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 weights4<float>(const float* p) { return __ldg(reinterpret_cast<const float4*>(p)); }
 template <>
 __device__ __forceinline__ float4 weights4<bf16>(const bf16* p) {
-    const uint2 q = *reinterpret_cast<const uint2*>(p);
+    const uint2 q = __ldg(reinterpret_cast<const uint2*>(p));
     const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
     return make_float4(lo.x, lo.y, hi.x, hi.y);
 }
@@ -341,10 +345,69 @@ struct StepArgs {
     int requests, width, block, taps, num_slots;
 };
 
-template <typename O, typename W, bool VEC>
+// u of one channel for the STEP_ROWS requests from r0 on; every load of the channel is asked for ahead of the sums.
+template <int TAPS>
+__device__ __forceinline__ void step_convolution(const StepArgs& a, int r0, int count, int c, const int* slot_s, float (&u)[STEP_ROWS]) {
+    const int taps = TAPS > 0 ? TAPS : a.taps;
+    const float bias = __ldg(a.bias + c), in_bias = __ldg(a.in_bias + c);
+    const float* w = a.taps_w + (long)c * taps;
+    float x[STEP_ROWS];
+#pragma unroll
+    for (int r = 0; r < STEP_ROWS; ++r) x[r] = r < count ? a.rows[(r0 + r) * a.row_stride + a.width + c] + in_bias : 0.0f;
+    if (TAPS > 0) {
+        float past[STEP_ROWS][TAPS > 1 ? TAPS - 1 : 1];
+#pragma unroll
+        for (int r = 0; r < STEP_ROWS; ++r) {
+            const int slot = r < count ? slot_s[r0 + r] : -1;
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j)
+                past[r][j] = slot >= 0 ? a.state[(long)slot * a.state_len + a.conv_off + (long)j * a.width + c] : 0.0f;
+        }
+#pragma unroll
+        for (int r = 0; r < STEP_ROWS; ++r) {
+            float acc = bias;
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) acc = fmaf(__ldg(w + j), past[r][j], acc);
+            u[r] = fmaf(__ldg(w + TAPS - 1), x[r], acc);
+        }
+    } else {
+#pragma unroll
+        for (int r = 0; r < STEP_ROWS; ++r) {
+            const int slot = r < count ? slot_s[r0 + r] : -1;
+            float acc = bias;
+            for (int j = 0; slot >= 0 && j + 1 < taps; ++j)
+                acc = fmaf(w[j], a.state[(long)slot * a.state_len + a.conv_off + (long)j * a.width + c], acc);
+            u[r] = fmaf(w[taps - 1], x[r], acc);
+        }
+    }
+}
+
+// 2 * ROWS sums over 32 lanes: halves change hands until a lane holds one sum's share (lane bits from the highest say which
+// sum), then the lanes that are left of it add up.
+template <int SUMS>
+__device__ __forceinline__ float fold_sums(float (&sum)[SUMS], int lane) {
+    int lanes = 16;
+#pragma unroll
+    for (int half = SUMS / 2; half >= 1; half >>= 1) {
+        const bool upper = (lane & lanes) != 0;
+#pragma unroll
+        for (int r = 0; r < half; ++r) {
+            const float give = upper ? sum[r] : sum[half + r];
+            const float got = __shfl_xor_sync(0xffffffffu, give, lanes);
+            sum[r] = (upper ? sum[half + r] : sum[r]) + got;
+        }
+        lanes >>= 1;
+    }
+    float total = sum[0];
+    for (; lanes >= 1; lanes >>= 1) total += __shfl_xor_sync(0xffffffffu, total, lanes);
+    return total;
+}
+
+template <typename O, typename W, bool VEC, int TAPS>
 __global__ void __launch_bounds__(256) real_gated_step_kernel(StepArgs a, O* __restrict__ out) {
     pdl_launch_dependents();
     extern __shared__ float step_smem[];
+    __shared__ int slot_s[STEP_REQUESTS];
     const int d = a.block, cuts = gridDim.x, b = blockIdx.y;
     const int per = (d + cuts - 1) / cuts;
     const int lo = min(d, (int)blockIdx.x * per), hi = min(d, lo + per);
@@ -358,24 +421,29 @@ __global__ void __launch_bounds__(256) real_gated_step_kernel(StepArgs a, O* __r
         const size_t bytes = (size_t)(hi - lo) * d * sizeof(W);
         for (size_t at = threadIdx.x * 128u; at < bytes; at += blockDim.x * 128u) asm volatile("prefetch.global.L2 [%0];" ::"l"(from + at));
     }
+    for (int r = threadIdx.x; r < a.requests; r += blockDim.x) {
+        const int slot = a.slots[r];
+        slot_s[r] = slot < a.num_slots ? slot : -1;
+    }
+    __syncthreads();
     pdl_wait();
-    const int taps = a.taps, width = a.width;
+    const int taps = TAPS > 0 ? TAPS : a.taps, width = a.width, own = hi - lo;
+    const RealGatedForm<O> form{nullptr, nullptr, 0, 0, d, nullptr, 0, a.r_bias, a.i_bias, a.branch_bias, a.rate, a.factor, out, a.out_stride, width};
     for (int r0 = 0; r0 < a.requests; r0 += STEP_ROWS) {
         const int count = min(STEP_ROWS, a.requests - r0);
         if (r0) __syncthreads();
-        for (int at = threadIdx.x; at < STEP_ROWS * d; at += blockDim.x) {
-            const int r = at / d, c = b * d + (at - r * d);
-            float acc = 0.0f;
-            if (r < count) {
-                const int slot = a.slots[r0 + r];
-                if (slot >= 0 && slot < a.num_slots) {
-                    const float* kept = a.state + (long)slot * a.state_len + a.conv_off + c;
-                    acc = a.bias[c];
-                    for (int j = 0; j + 1 < taps; ++j) acc = fmaf(a.taps_w[(long)c * taps + j], kept[(long)j * width], acc);
-                    acc = fmaf(a.taps_w[(long)c * taps + taps - 1], a.rows[(r0 + r) * a.row_stride + width + c] + a.in_bias[c], acc);
-                }
-            }
-            u_s[at] = acc;
+        for (int j = threadIdx.x; j < d; j += blockDim.x) {
+            float u[STEP_ROWS];
+            step_convolution<TAPS>(a, r0, count, b * d + j, slot_s, u);
+#pragma unroll
+            for (int r = 0; r < STEP_ROWS; ++r) u_s[r * d + j] = u[r];
+        }
+        // the first (request, channel) that this thread will finish: its state and branch are asked for here
+        float first_s = 0.0f, first_branch = 0.0f;
+        if (threadIdx.x < count * own) {
+            const int r = threadIdx.x / own, c = b * d + lo + threadIdx.x - r * own, slot = slot_s[r0 + r];
+            if (slot >= 0) first_s = a.state[(long)slot * a.state_len + a.state_off + c];
+            first_branch = a.rows[(r0 + r) * a.row_stride + c];
         }
         __syncthreads();
         for (int j = lo + warp; j < hi; j += warps) {
@@ -385,13 +453,25 @@ __global__ void __launch_bounds__(256) real_gated_step_kernel(StepArgs a, O* __r
 #pragma unroll
             for (int r = 0; r < 2 * STEP_ROWS; ++r) sum[r] = 0.0f;
             if (VEC) {
-                for (int k = lane * 4; k < d; k += 128) {
-                    const float4 wr = weights4<W>(row_r + k), wi = weights4<W>(row_i + k);
+                for (int k0 = lane * 4; k0 < d; k0 += 256) {
+                    // two pieces' weights at once
+                    const int k1 = k0 + 128;
+                    const float4 none = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                    const float4 wr0 = weights4<W>(row_r + k0), wi0 = weights4<W>(row_i + k0);
+                    const float4 wr1 = k1 < d ? weights4<W>(row_r + k1) : none, wi1 = k1 < d ? weights4<W>(row_i + k1) : none;
 #pragma unroll
                     for (int r = 0; r < STEP_ROWS; ++r) {
-                        const float4 u = *reinterpret_cast<const float4*>(u_s + r * d + k);
-                        sum[r] = fmaf(wr.x, u.x, fmaf(wr.y, u.y, fmaf(wr.z, u.z, fmaf(wr.w, u.w, sum[r]))));
-                        sum[STEP_ROWS + r] = fmaf(wi.x, u.x, fmaf(wi.y, u.y, fmaf(wi.z, u.z, fmaf(wi.w, u.w, sum[STEP_ROWS + r]))));
+                        const float4 u = *reinterpret_cast<const float4*>(u_s + r * d + k0);
+                        sum[r] = fmaf(wr0.x, u.x, fmaf(wr0.y, u.y, fmaf(wr0.z, u.z, fmaf(wr0.w, u.w, sum[r]))));
+                        sum[STEP_ROWS + r] = fmaf(wi0.x, u.x, fmaf(wi0.y, u.y, fmaf(wi0.z, u.z, fmaf(wi0.w, u.w, sum[STEP_ROWS + r]))));
+                    }
+                    if (k1 < d) {
+#pragma unroll
+                        for (int r = 0; r < STEP_ROWS; ++r) {
+                            const float4 u = *reinterpret_cast<const float4*>(u_s + r * d + k1);
+                            sum[r] = fmaf(wr1.x, u.x, fmaf(wr1.y, u.y, fmaf(wr1.z, u.z, fmaf(wr1.w, u.w, sum[r]))));
+                            sum[STEP_ROWS + r] = fmaf(wi1.x, u.x, fmaf(wi1.y, u.y, fmaf(wi1.z, u.z, fmaf(wi1.w, u.w, sum[STEP_ROWS + r]))));
+                        }
                     }
                 }
             } else {
@@ -404,36 +484,22 @@ __global__ void __launch_bounds__(256) real_gated_step_kernel(StepArgs a, O* __r
                     }
                 }
             }
-            // sixteen sums over 32 lanes: halves change hands until a lane holds one sum, then the last two lanes add up
-#pragma unroll
-            for (int half = STEP_ROWS, lanes = 16; half >= 1; half >>= 1, lanes >>= 1) {
-                const bool upper = (lane & lanes) != 0;
-#pragma unroll
-                for (int r = 0; r < half; ++r) {
-                    const float give = upper ? sum[r] : sum[half + r];
-                    const float got = __shfl_xor_sync(0xffffffffu, give, lanes);
-                    sum[r] = (upper ? sum[half + r] : sum[r]) + got;
-                }
-            }
-            const float total = sum[0] + __shfl_xor_sync(0xffffffffu, sum[0], 1);
-            // lane bits 4, 3, 2, 1 say which sum it is, the highest first
-            const int which = lane >> 1;
-            if ((lane & 1) == 0) gate_s[which * per + (j - lo)] = total;
+            const float total = fold_sums<2 * STEP_ROWS>(sum, lane);
+            if ((lane & 1) == 0) gate_s[(lane >> 1) * per + (j - lo)] = total;
         }
         __syncthreads();
-        for (int at = threadIdx.x; at < count * (hi - lo); at += blockDim.x) {
-            const int r = at / (hi - lo), j = at - r * (hi - lo);
-            const int slot = a.slots[r0 + r];
-            if (slot < 0 || slot >= a.num_slots) continue;
+        for (int at = threadIdx.x; at < count * own; at += blockDim.x) {
+            const int r = at / own, j = at - r * own, slot = slot_s[r0 + r];
+            if (slot < 0) continue;
             const int c = b * d + lo + j;
-            const RealGatedForm<O> form{nullptr, nullptr, 0, 0, d, nullptr, 0, a.r_bias, a.i_bias, a.branch_bias, a.rate, a.factor, out, a.out_stride, width};
+            float* S = a.state + (long)slot * a.state_len + a.state_off + c;
+            const bool held = at == (int)threadIdx.x;
             const typename RealGatedForm<O>::Channel ch = form.channel(c);
             const typename RealGatedForm<O>::Row row{gate_s[r * per + j], gate_s[(STEP_ROWS + r) * per + j], u_s[r * d + lo + j],
-                                                     a.rows[(r0 + r) * a.row_stride + c]};
-            float* S = a.state + (long)slot * a.state_len + a.state_off + c;
+                                                     held ? first_branch : a.rows[(r0 + r) * a.row_stride + c]};
             float keep, take;
             form.terms(ch, row, keep, take);
-            const float s = fmaf(keep, *S, take);
+            const float s = fmaf(keep, held ? first_s : *S, take);
             *S = s;
             form.store(ch, form.keep(row), r0 + r, s);
         }
@@ -441,10 +507,9 @@ __global__ void __launch_bounds__(256) real_gated_step_kernel(StepArgs a, O* __r
     // every CTA of the cluster has read the block's kept rows
     asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
     if (taps > 1) {
-        for (int at = threadIdx.x; at < a.requests * (hi - lo); at += blockDim.x) {
-            const int r = at / (hi - lo), c = b * d + lo + (at - r * (hi - lo));
-            const int slot = a.slots[r];
-            if (slot < 0 || slot >= a.num_slots) continue;
+        for (int at = threadIdx.x; at < a.requests * own; at += blockDim.x) {
+            const int r = at / own, c = b * d + lo + (at - r * own), slot = slot_s[r];
+            if (slot < 0) continue;
             float* kept = a.state + (long)slot * a.state_len + a.conv_off + c;
             for (int k = 0; k + 2 < taps; ++k) kept[(long)k * width] = kept[(long)(k + 1) * width];
             kept[(long)(taps - 2) * width] = a.rows[r * a.row_stride + width + c] + a.in_bias[c];
@@ -452,9 +517,16 @@ __global__ void __launch_bounds__(256) real_gated_step_kernel(StepArgs a, O* __r
     }
 }
 
+template <typename O, typename W, bool VEC>
+void (*step_kernel(int taps))(StepArgs, O*) {
+    return taps == 2 ? real_gated_step_kernel<O, W, VEC, 2> : taps == 3 ? real_gated_step_kernel<O, W, VEC, 3>
+         : taps == 4 ? real_gated_step_kernel<O, W, VEC, 4> : real_gated_step_kernel<O, W, VEC, 0>;
+}
+
 template <typename O>
 int real_gated_step_launch(const StepArgs& a, int gates_bf16, void* out, cudaStream_t stream) {
     if (a.requests <= 0) return 0;
+    if (a.requests > STEP_REQUESTS) return KIRAI_ERR_BAD_SIZE;
     if (a.width <= 0 || a.block <= 0 || a.width % a.block || a.taps < 1 || a.conv_off < 0 || a.state_off < 0 || a.out_stride < a.width ||
         a.conv_off + (long)(a.taps - 1) * a.width > a.state_len || a.state_off + a.width > a.state_len)
         return KIRAI_ERR_BAD_SIZE;
@@ -466,8 +538,8 @@ int real_gated_step_launch(const StepArgs& a, int gates_bf16, void* out, cudaStr
     const size_t smem = (size_t)STEP_ROWS * (a.block + 2 * per) * sizeof(float);
     if (smem > 200 * 1024) return KIRAI_ERR_BAD_SIZE;
     const bool vec = a.block % 4 == 0 && ((uintptr_t)a.gates & 15) == 0;
-    auto kernel = gates_bf16 ? (vec ? real_gated_step_kernel<O, bf16, true> : real_gated_step_kernel<O, bf16, false>)
-                             : (vec ? real_gated_step_kernel<O, float, true> : real_gated_step_kernel<O, float, false>);
+    auto kernel = gates_bf16 ? (vec ? step_kernel<O, bf16, true>(a.taps) : step_kernel<O, bf16, false>(a.taps))
+                             : (vec ? step_kernel<O, float, true>(a.taps) : step_kernel<O, float, false>(a.taps));
     if (smem > 48 * 1024) {
         const cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (err != cudaSuccess) return (int)err;
@@ -495,20 +567,24 @@ KIRAI_REAL_GATED_STEP(kirai_real_gated_step_bf16, bf16)
 
 // out [T, channels] (float32) = (silu of) bias + sum_j taps_w[c, j] * (in[t - (taps - 1) + j, c] + in_bias[c]) per request,
 // kept rows before a request's first row of this step; then the kept rows move on.  pair (may be null): the same rows as
-// high and low bfloat16 parts, [channels / block, pair_tokens, 2 block].
+// high and low bfloat16 parts, [channels / block, pair_tokens, 2 block].  single: every request brings one token.
 KIRAI_EXPORT int kirai_conv_rows(const float* in, long in_stride, const float* taps_w, const float* in_bias, const float* bias,
                                  float* state, long state_len, long conv_off, const int* request_of_token, const int* query_start,
-                                 const int* slots, float* out, void* pair, int block, int pair_tokens, int silu, int tokens,
-                                 int requests, int channels, int taps, int num_slots, cudaStream_t stream) {
+                                 const int* slots, float* out, void* pair, int block, int pair_tokens, int silu, int single,
+                                 int tokens, int requests, int channels, int taps, int num_slots, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (channels <= 0 || taps <= 0 || requests <= 0 || conv_off < 0 || conv_off + (long)(taps - 1) * channels > state_len)
         return KIRAI_ERR_BAD_SIZE;
     if (pair && (block <= 0 || channels % block || pair_tokens < tokens)) return KIRAI_ERR_BAD_SIZE;
-    const ConvArgs a{in, in_stride, taps_w, in_bias, bias, state, state_len, conv_off, request_of_token, query_start, slots, out,
-                     (bf16*)pair, block, pair_tokens, tokens, channels, num_slots, silu};
     const int threads = channels >= 8192 || tokens >= 512 ? 256 : 128;
     const unsigned columns = (unsigned)((channels + threads - 1) / threads);
-    const unsigned walks = (unsigned)((tokens + CONV_RUN - 1) / CONV_RUN);
+    // few tokens: shorter runs, so that more blocks ask for rows at the same time
+    int run = CONV_RUN;
+    while (run > 1 && (long)((tokens + run - 1) / run) * columns < 592) run >>= 1;
+    if (single) run = 1;
+    const ConvArgs a{in, in_stride, taps_w, in_bias, bias, state, state_len, conv_off, request_of_token, query_start, slots, out,
+                     (bf16*)pair, block, pair_tokens, tokens, channels, num_slots, silu, run, single && taps <= 4};
+    const unsigned walks = (unsigned)((tokens + run - 1) / run);
     int status;
     switch (taps) {
         case 1: status = launch_pdl(conv_run_kernel<1>, dim3(walks, columns), dim3(threads), 0, stream, 1u, a); break;
@@ -517,7 +593,7 @@ KIRAI_EXPORT int kirai_conv_rows(const float* in, long in_stride, const float* t
         case 4: status = launch_pdl(conv_run_kernel<4>, dim3(walks, columns), dim3(threads), 0, stream, 1u, a); break;
         default: status = launch_pdl(conv_any_kernel, dim3(tokens, columns), dim3(threads), 0, stream, 1u, a, taps); break;
     }
-    if (status != 0 || taps == 1) return status;
+    if (status != 0 || taps == 1 || a.single) return status;
     const long units = (long)requests * channels;
     return launch_pdl(conv_keep_kernel, dim3((unsigned)((units + 255) / 256)), dim3(256), 0, stream, 1u, in, in_stride, in_bias, state,
                       state_len, conv_off, query_start, slots, requests, channels, taps, num_slots);

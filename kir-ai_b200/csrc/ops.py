@@ -725,7 +725,7 @@ def conv_rows(x: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tensor],
         pair = torch.empty((channels // pair_block, pair_tokens, 2 * pair_block), dtype=torch.bfloat16, device=x.device)
     _call("kirai_conv_rows", _ptr(x), _l(x.stride(0)), _ptr(taps), _ptr(in_bias), _ptr(bias), _ptr(state), _l(state.shape[1]),
           _l(conv_offset), _ptr(batch.request_of_token), _ptr(batch.query_start), _ptr(batch.slots), _ptr(out), _ptr(pair),
-          _i(pair_block), _i(pair_tokens), _i(int(silu)), _i(x.shape[0]), _i(batch.num_requests), _i(channels), _i(width),
+          _i(pair_block), _i(pair_tokens), _i(int(silu)), _i(int(batch.decode_only)), _i(x.shape[0]), _i(batch.num_requests), _i(channels), _i(width),
           _i(state.shape[0]), _stream(), detail=f" c={channels}" if _timer is not None else "")
     return (out, pair) if pair_block else out
 
