@@ -22,15 +22,29 @@ import torch
 
 
 @dataclass(frozen=True)
+class OpenSize:
+    """A size that no configuration gives: the stored tensors' own, the same wherever ``name`` stands.  ``default`` is
+    what the random-weights mode takes."""
+
+    name: str
+    default: int
+
+
+@dataclass(frozen=True)
 class WeightSpec:
     """Shape and role of one named tensor.  The role tells the random-weights
     mode how to fill it and the loader which dtype family it must have:
     ``linear`` and ``embedding`` are floating matrices, ``norm`` a floating
     vector around one, ``bias`` a floating vector around zero, ``identity`` a square matrix
-    around the identity, ``int_table`` an integer table (kept as int32)."""
+    around the identity, ``int_table`` an integer table (kept as int32).  An entry of ``shape`` is a number or an
+    ``OpenSize``."""
 
-    shape: Tuple[int, ...]
+    shape: Tuple[object, ...]
     role: str = "linear"
+
+    def sizes(self) -> Tuple[int, ...]:
+        """The shape with every open size at its default."""
+        return tuple(s.default if isinstance(s, OpenSize) else s for s in self.shape)
 
 
 @dataclass(frozen=True)

@@ -19,7 +19,7 @@ from typing import Dict, Mapping, Optional
 
 import torch
 
-from ..parts.base import WeightSpec
+from ..parts.base import OpenSize, WeightSpec
 from .safetensors_io import ModelFiles
 
 _FLOAT = {"F32", "BF16", "F16", "F64"}
@@ -89,13 +89,19 @@ def check(specs: Mapping[str, WeightSpec], present: Mapping[str, tuple], ignorab
     reference, which only asks for the names it needs (crates/llm-models/src/qwen.rs:215-260)."""
     missing = [name for name in specs if name not in present]
     unexpected = [name for name in present if name not in specs and name not in set(ignorable)]
-    wrong = []
+    wrong, open_sizes = [], {}
     for name, spec in specs.items():
         if name not in present:
             continue
         dtype, shape = present[name]
-        if tuple(shape) != tuple(spec.shape):
-            wrong.append(f"{name}: shape {list(shape)}, expected {list(spec.shape)}")
+        # an open size is whatever the first tensor that has it says; every other must agree
+        expected = list(spec.shape)
+        for axis, size in enumerate(expected):
+            if isinstance(size, OpenSize):
+                fits = len(shape) == len(expected) and shape[axis] > 0
+                expected[axis] = open_sizes.setdefault(size.name, shape[axis]) if fits else open_sizes.get(size.name, size.name)
+        if list(shape) != expected:
+            wrong.append(f"{name}: shape {list(shape)}, expected {expected}")
         elif spec.role == "int_table" and dtype not in _INT:
             wrong.append(f"{name}: dtype {dtype}, expected an integer table")
         elif spec.role != "int_table" and dtype not in _FLOAT:

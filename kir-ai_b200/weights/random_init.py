@@ -38,13 +38,13 @@ def random_tensors(specs: Mapping[str, WeightSpec], seed: int, *, std: float = 0
     for name, spec in specs.items():
         generator = _generator(seed, name, device)
         if spec.role == "int_table":
-            tensors[name] = torch.randint(0, int_table_range, spec.shape, generator=generator, device=device, dtype=torch.int32)
+            tensors[name] = torch.randint(0, int_table_range, spec.sizes(), generator=generator, device=device, dtype=torch.int32)
             continue
-        values = torch.randn(spec.shape, generator=generator, device=device, dtype=torch.float32)
+        values = torch.randn(spec.sizes(), generator=generator, device=device, dtype=torch.float32)
         if spec.role == "norm":
             values = 1.0 + norm_jitter * values
         elif spec.role == "identity":
-            values = torch.eye(spec.shape[0], device=device) + norm_jitter * values
+            values = torch.eye(spec.sizes()[0], device=device) + norm_jitter * values
         else:
             values = std * values
         tensors[name] = values.to(dtype)
