@@ -27,6 +27,8 @@ SOURCES = [
     "mixer_forms.cu",
     "state_forms.cu",
     "state_chunks.cu",
+    "channel_scan.cu",
+    "token_forms.cu",
     "gated_scan.cu",
     "stream_forms.cu",
     "experts.cu",
@@ -39,7 +41,7 @@ SOURCES = [
     "attention_tcgen05.cu",
     "wait_selftest.cu",
 ]
-HEADERS = ["common.cuh", "state_math.cuh", "sm100.cuh", "tensor_map.cuh", "no_alloc.h"]
+HEADERS = ["common.cuh", "state_math.cuh", "chunk_tiles.cuh", "sm100.cuh", "tensor_map.cuh", "no_alloc.h"]
 
 NVCC_FLAGS = [
     "-gencode",

@@ -6,8 +6,12 @@
 //                  experts' shares of the softmax over ALL logits, which then do not sum to one; or, with rule 2, sigmoid
 //                  scores: the choice looks at sigmoid(z) + correction, and only inside the `keep` of `groups` equal
 //                  groups of neighbouring experts whose two largest such numbers sum highest, and the weights are
-//                  the chosen experts' sigmoid(z) as they are).  The result is the dense matrix
-//                  gates [T, experts], zero where an expert was not chosen, plus the chosen ids and weights.
+//                  the chosen experts' sigmoid(z) as they are; rule 3: scores are the softmax over all, the choice
+//                  looks at score + correction, the weights are the chosen scores divided by their sum (+ 1e-20), times
+//                  `scale`).  The result is the dense matrix
+//                  gates [T, experts], zero where an expert was not chosen, plus the chosen ids and weights.  `extra`
+//                  further rows of the matrix may stand behind the experts': their logits come out as sigmoid(z), in
+//                  columns behind the experts'.
 //   relu2_gate     hidden[t, e * ff + j] = relu(up[t, e * ff + j])^2 * gates[t, e]: with the experts' up matrices
 //                  stacked along the rows and their down matrices side by side along the columns, the product
 //                  hidden W_down^T is the weighted sum of the chosen experts' outputs, and an expert that was not
@@ -31,11 +35,14 @@ __device__ __forceinline__ float4 load4(const bf16* p) {
 // [experts] of logits (read past L1), picks the `top` largest one after the other (the lower index wins a tie) and
 // overwrites the row with the routing weights.  `logits_s` [experts] is this warp's shared scratch.
 // How the weights come from the logits.  mode 0: softmax over the chosen logits; 1: the chosen experts' shares of the
-// softmax over all; 2: sigmoid scores with a correction on the choice and a choice among groups (see the top of the file).
+// softmax over all; 2: sigmoid scores with a correction on the choice and a choice among groups; 3: softmax scores with a
+// correction on the choice, the chosen ones brought to the sum `scale` (see the top of the file).
 struct RouterRule {
     int mode;
-    const float* correction;  // [experts] or null (mode 2)
+    const float* correction;  // [experts] or null (modes 2 and 3)
     int groups, keep;         // mode 2; one group of which one is kept: no limit
+    float scale;              // mode 3
+    int extra;                // columns behind the experts' that become sigmoid(z)
 };
 // Floats of shared scratch a warp needs to choose for one token: logits, scores, group scores.
 #define ROUTER_SCRATCH(experts) (3 * (size_t)(experts))
@@ -44,16 +51,26 @@ __device__ __forceinline__ void choose_experts(float* __restrict__ out, float* l
                                                float* __restrict__ chosen_weights, int experts, int top, int lane,
                                                const RouterRule rule) {
     const int over_all = rule.mode == 1;
-    const bool scored = rule.mode == 2;
-    float* scores_s = logits_s + experts;       // mode 2: sigmoid(z), the weights
+    const bool scored = rule.mode == 2 || rule.mode == 3;
+    float* scores_s = logits_s + experts;       // modes 2 and 3: the scores, from which the weights come
     float* groups_s = logits_s + 2 * experts;   // mode 2: every group's two largest choice scores, summed
     for (int i = lane; i < experts; i += 32) logits_s[i] = __ldcg(out + i);
     __syncwarp();
     for (int i = lane; i < experts; i += 32) out[i] = 0.0f;
+    for (int i = lane; i < rule.extra; i += 32) out[experts + i] = 1.0f / (1.0f + expf(-__ldcg(out + experts + i)));
     __syncwarp();
     if (scored) {
+        float top_logit = 0.0f, inverse = 0.0f;
+        if (rule.mode == 3) {
+            top_logit = -INFINITY;
+            for (int i = lane; i < experts; i += 32) top_logit = fmaxf(top_logit, logits_s[i]);
+            top_logit = warp_max(top_logit);
+            float sum = 0.0f;
+            for (int i = lane; i < experts; i += 32) sum += expf(logits_s[i] - top_logit);
+            inverse = 1.0f / warp_sum(sum);
+        }
         for (int i = lane; i < experts; i += 32) {
-            const float score = 1.0f / (1.0f + expf(-logits_s[i]));
+            const float score = rule.mode == 3 ? expf(logits_s[i] - top_logit) * inverse : 1.0f / (1.0f + expf(-logits_s[i]));
             scores_s[i] = score;
             logits_s[i] = score + (rule.correction ? rule.correction[i] : 0.0f);  // what the choice looks at
         }
@@ -129,7 +146,7 @@ __device__ __forceinline__ void choose_experts(float* __restrict__ out, float* l
     }
     __syncwarp();
     if (over_all) denom = all_sum;  // (the first chosen logit is the maximum of all)
-    const float inv = scored ? 1.0f : (denom > 0.0f ? 1.0f / denom : 0.0f);
+    const float inv = rule.mode == 3 ? rule.scale / (denom + 1e-20f) : scored ? 1.0f : (denom > 0.0f ? 1.0f / denom : 0.0f);
     for (int i = lane; i < experts; i += 32) out[i] *= inv;
     if (chosen_weights)
         for (int k = lane; k < top; k += 32) chosen_weights[k] *= inv;
@@ -167,7 +184,7 @@ router_gates_few_kernel(const T* __restrict__ x, long x_stride, const float* __r
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const T* row = x + (size_t)token * x_stride;
     const float* w = router + (size_t)e * hidden;
-    float* out = gates + (size_t)token * experts;
+    float* out = gates + (size_t)token * (experts + rule.extra);
     float dot = 0.0f;
     if (hidden % 4 == 0 && x_stride % 4 == 0 && (((uintptr_t)x | (uintptr_t)router) & 15) == 0) {
         float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
@@ -210,7 +227,7 @@ router_gates_many_kernel(const T* __restrict__ x, long x_stride, const float* __
     const int count = min(ROUTER_TOKENS, tokens - first);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int e = blockIdx.y * ROUTER_WARPS + warp;
-    if (e < experts) {
+    if (e < experts + rule.extra) {
         const float* w = router + (size_t)e * hidden;
         float dot[ROUTER_TOKENS];
 #pragma unroll
@@ -238,20 +255,20 @@ router_gates_many_kernel(const T* __restrict__ x, long x_stride, const float* __
 #pragma unroll
         for (int t = 0; t < ROUTER_TOKENS; ++t) {
             const float total = warp_sum(dot[t]);
-            if (lane == 0 && t < count) gates[(size_t)(first + t) * experts + e] = total;
+            if (lane == 0 && t < count) gates[(size_t)(first + t) * (experts + rule.extra) + e] = total;
         }
     }
     if (!arrives_last(&arrivals[blockIdx.x], (int)gridDim.y, &is_last)) return;
     for (int t = warp; t < count; t += ROUTER_WARPS) {
         const size_t token = (size_t)(first + t);
-        choose_experts(gates + token * experts, logits_s + warp * ROUTER_SCRATCH(experts), chosen_ids ? chosen_ids + token * top : nullptr,
+        choose_experts(gates + token * (experts + rule.extra), logits_s + warp * ROUTER_SCRATCH(experts), chosen_ids ? chosen_ids + token * top : nullptr,
                        chosen_weights ? chosen_weights + token * top : nullptr, experts, top, lane, rule);
     }
 }
 
 // Whether a rule fits the experts it is to choose among.
 static bool router_rule_fits(const RouterRule& rule, int experts, int top) {
-    if (rule.mode < 0 || rule.mode > 2) return false;
+    if (rule.mode < 0 || rule.mode > 3 || rule.extra < 0 || rule.extra > 32) return false;
     if (rule.mode != 2) return true;
     if (rule.groups <= 0 || rule.keep <= 0 || rule.keep > rule.groups || experts % rule.groups != 0) return false;
     return top <= rule.keep * (experts / rule.groups);
@@ -265,11 +282,12 @@ static int router_gates_launch(const void* x, long x_stride, const float* router
     if (experts <= 0 || top <= 0 || top > experts || hidden <= 0 || experts > 1024 || !arrivals) return KIRAI_ERR_BAD_SIZE;
     if (!router_rule_fits(rule, experts, top)) return KIRAI_ERR_BAD_SIZE;
     if ((chosen_ids == nullptr) != (chosen_weights == nullptr)) return KIRAI_ERR_BAD_SIZE;
-    if (tokens * (long)experts <= 4096 && experts <= 65535) {
-        return launch_pdl(router_gates_few_kernel<T>, dim3(tokens, experts), dim3(ROUTER_WARPS * 32), ROUTER_SCRATCH(experts) * sizeof(float),
+    const int columns = experts + rule.extra;
+    if (tokens * (long)columns <= 4096) {
+        return launch_pdl(router_gates_few_kernel<T>, dim3(tokens, columns), dim3(ROUTER_WARPS * 32), ROUTER_SCRATCH(experts) * sizeof(float),
                           stream, 1u, (const T*)x, x_stride, router, gates, chosen_ids, chosen_weights, arrivals, hidden, experts, top, rule);
     }
-    const unsigned slices = (unsigned)((experts + ROUTER_WARPS - 1) / ROUTER_WARPS);
+    const unsigned slices = (unsigned)((columns + ROUTER_WARPS - 1) / ROUTER_WARPS);
     const unsigned groups = (unsigned)((tokens + ROUTER_TOKENS - 1) / ROUTER_TOKENS);
     return launch_pdl(router_gates_many_kernel<T>, dim3(groups, slices), dim3(ROUTER_WARPS * 32),
                       ROUTER_WARPS * ROUTER_SCRATCH(experts) * sizeof(float), stream, 1u, (const T*)x, x_stride, router, gates, chosen_ids,
@@ -286,18 +304,18 @@ router_choose_kernel(float* __restrict__ gates, int* __restrict__ chosen_ids, fl
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const size_t token = (size_t)blockIdx.x * ROUTER_WARPS + warp;
     if (token >= (size_t)tokens) return;
-    choose_experts(gates + token * experts, logits_s + warp * ROUTER_SCRATCH(experts), chosen_ids ? chosen_ids + token * top : nullptr,
+    choose_experts(gates + token * (experts + rule.extra), logits_s + warp * ROUTER_SCRATCH(experts), chosen_ids ? chosen_ids + token * top : nullptr,
                    chosen_weights ? chosen_weights + token * top : nullptr, experts, top, lane, rule);
 }
 
 // gates [tokens, experts] holds router logits (32-bit) and receives the routing weights; see router_gates.
-// rule, correction, groups, keep: see RouterRule.
+// rule, correction, groups, keep, scale, extra: see RouterRule.  Rows have experts + extra numbers.
 KIRAI_EXPORT int kirai_router_choose(float* gates, int* chosen_ids, float* chosen_weights, int tokens, int experts, int top,
-                                     int rule, const float* correction, int groups, int keep, cudaStream_t stream) {
+                                     int rule, const float* correction, int groups, int keep, float scale, int extra, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (experts <= 0 || top <= 0 || top > experts || experts > 1024) return KIRAI_ERR_BAD_SIZE;
     if ((chosen_ids == nullptr) != (chosen_weights == nullptr)) return KIRAI_ERR_BAD_SIZE;
-    const RouterRule how{rule, correction, groups, keep};
+    const RouterRule how{rule, correction, groups, keep, scale, extra};
     if (!router_rule_fits(how, experts, top)) return KIRAI_ERR_BAD_SIZE;
     return launch_pdl(router_choose_kernel, dim3((unsigned)((tokens + ROUTER_WARPS - 1) / ROUTER_WARPS)), dim3(ROUTER_WARPS * 32),
                       ROUTER_WARPS * ROUTER_SCRATCH(experts) * sizeof(float), stream, 1u, gates, chosen_ids, chosen_weights, tokens, experts, top, how);
@@ -306,15 +324,15 @@ KIRAI_EXPORT int kirai_router_choose(float* gates, int* chosen_ids, float* chose
 // arrivals [tokens]: zero before the first launch; every launch leaves it zero.
 KIRAI_EXPORT int kirai_router_gates_f32(const void* x, long x_stride, const float* router, float* gates, int* chosen_ids,
                                         float* chosen_weights, int* arrivals, int tokens, int hidden, int experts, int top,
-                                        int rule, const float* correction, int groups, int keep, cudaStream_t stream) {
+                                        int rule, const float* correction, int groups, int keep, float scale, int extra, cudaStream_t stream) {
     return router_gates_launch<float>(x, x_stride, router, gates, chosen_ids, chosen_weights, arrivals, tokens, hidden, experts, top,
-                                      RouterRule{rule, correction, groups, keep}, stream);
+                                      RouterRule{rule, correction, groups, keep, scale, extra}, stream);
 }
 KIRAI_EXPORT int kirai_router_gates_bf16(const void* x, long x_stride, const float* router, float* gates, int* chosen_ids,
                                          float* chosen_weights, int* arrivals, int tokens, int hidden, int experts, int top,
-                                         int rule, const float* correction, int groups, int keep, cudaStream_t stream) {
+                                         int rule, const float* correction, int groups, int keep, float scale, int extra, cudaStream_t stream) {
     return router_gates_launch<bf16>(x, x_stride, router, gates, chosen_ids, chosen_weights, arrivals, tokens, hidden, experts, top,
-                                     RouterRule{rule, correction, groups, keep}, stream);
+                                     RouterRule{rule, correction, groups, keep, scale, extra}, stream);
 }
 
 // activation: 0 = relu(z)^2
@@ -546,4 +564,157 @@ KIRAI_EXPORT int kirai_route_combine_norm_add_bf16(float* resid, const void* y, 
     const int threads = hidden <= 4 * 4 * 128 ? 128 : (hidden <= 4 * 4 * 256 ? 256 : 512);
     return launch_pdl(route_combine_norm_add_kernel<4>, dim3(tokens), dim3(threads), 0, stream, 1u, resid, (const bf16*)y, slot_of,
                       weights, norm_weight, (bf16*)copy, hidden, top, eps);
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// What a feed-forward of several terms adds up to, and the norm on its output:
+//
+//     y = routed + sum_j weight_j sorted[slot_j] + share shared + same stream
+//
+// `routed` [T, H] (32-bit) or rows sorted by expert with their slots and weights (either may be missing), `shared` [T, H]
+// (32-bit) a branch that every token runs, `share` its weight (number `share_col` of the token's row of `gates`; 1 when
+// share_col < 0), and `same` the sum of `same_count` numbers of that row from `same_col`: the weight of experts that hand
+// their input on, which is the stream itself.  The stream takes y * rsqrt(mean(y^2) + eps) * norm_weight, and `copy` is the
+// new stream in bfloat16.  One block per token, the row in registers (width a multiple of 4, at most 4 VEC blockDim values).
+struct FeedForwardTerms {
+    const float* routed;
+    const bf16* sorted;
+    const int* slot_of;
+    const float* weights;
+    const float* shared;
+    const float* gates;
+    long gates_stride;
+    int top, share_col, same_col, same_count;
+};
+
+__device__ __forceinline__ float same_weight(const FeedForwardTerms& f, int token) {
+    float sum = 0.0f;
+    for (int i = 0; i < f.same_count; ++i) sum += f.gates[(size_t)token * f.gates_stride + f.same_col + i];
+    return sum;
+}
+
+__device__ __forceinline__ void add_scaled4(float4& to, float w, const float4 v) {
+    to.x = fmaf(w, v.x, to.x), to.y = fmaf(w, v.y, to.y), to.z = fmaf(w, v.z, to.z), to.w = fmaf(w, v.w, to.w);
+}
+
+template <int VEC>
+__global__ void terms_norm_add_kernel(float* __restrict__ resid, const FeedForwardTerms f, const float* __restrict__ norm_weight,
+                                      bf16* __restrict__ copy, int hidden, float eps) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float scratch[32];
+    const int token = blockIdx.x;
+    const int quads = hidden >> 2;
+    const size_t base = (size_t)token * hidden;
+    const float share = f.shared && f.share_col >= 0 ? f.gates[(size_t)token * f.gates_stride + f.share_col] : 1.0f;
+    const float same = same_weight(f, token);
+    float4* dst = reinterpret_cast<float4*>(resid + base);
+    float4 kept[VEC], stream[VEC];
+    float acc = 0.0f;
+#pragma unroll
+    for (int n = 0; n < VEC; ++n) {
+        const int i = threadIdx.x + n * blockDim.x;
+        kept[n] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (i < quads) {
+            stream[n] = dst[i];
+            if (f.routed) kept[n] = load4(f.routed + base + 4 * (size_t)i);
+            if (f.sorted) {
+                for (int j = 0; j < f.top; ++j) {
+                    const int slot = f.slot_of[(size_t)token * f.top + j];
+                    if (slot >= 0) add_scaled4(kept[n], f.weights[(size_t)token * f.top + j], load4(f.sorted + (size_t)slot * hidden + 4 * (size_t)i));
+                }
+            }
+            if (f.shared) add_scaled4(kept[n], share, load4(f.shared + base + 4 * (size_t)i));
+            if (same != 0.0f) add_scaled4(kept[n], same, stream[n]);
+            acc += (kept[n].x * kept[n].x + kept[n].y * kept[n].y) + (kept[n].z * kept[n].z + kept[n].w * kept[n].w);
+        }
+    }
+    const float variance = block_sum(acc, scratch) / (float)hidden + eps;
+    const float scale = variance == 0.0f ? 0.0f : 1.0f / sqrtf(variance);
+    const float4* w4 = reinterpret_cast<const float4*>(norm_weight);
+#pragma unroll
+    for (int n = 0; n < VEC; ++n) {
+        const int i = threadIdx.x + n * blockDim.x;
+        if (i < quads) {
+            float4 r = stream[n];
+            const float4 w = w4[i];
+            r.x += kept[n].x * scale * w.x, r.y += kept[n].y * scale * w.y, r.z += kept[n].z * scale * w.z, r.w += kept[n].w * scale * w.w;
+            dst[i] = r;
+            if (copy) {
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(r.x, r.y), hi = __floats2bfloat162_rn(r.z, r.w);
+                uint2 packed;
+                packed.x = *reinterpret_cast<const uint32_t*>(&lo);
+                packed.y = *reinterpret_cast<const uint32_t*>(&hi);
+                *reinterpret_cast<uint2*>(copy + base + 4 * (size_t)i) = packed;
+            }
+        }
+    }
+}
+
+// The sum alone, out [T, H] (32-bit), for any width; `input` [T, H] is what the experts read.
+template <typename T>
+__global__ void terms_sum_kernel(const FeedForwardTerms f, const T* __restrict__ input, long input_stride, float* __restrict__ out, int hidden) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int token = blockIdx.x;
+    const float share = f.shared && f.share_col >= 0 ? f.gates[(size_t)token * f.gates_stride + f.share_col] : 1.0f;
+    const float same = same_weight(f, token);
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        const size_t at = (size_t)token * hidden + i;
+        float sum = f.routed ? f.routed[at] : 0.0f;
+        if (f.sorted) {
+            for (int j = 0; j < f.top; ++j) {
+                const int slot = f.slot_of[(size_t)token * f.top + j];
+                if (slot >= 0) sum = fmaf(f.weights[(size_t)token * f.top + j], to_f32<bf16>(f.sorted[(size_t)slot * hidden + i]), sum);
+            }
+        }
+        if (f.shared) sum = fmaf(share, f.shared[at], sum);
+        if (same != 0.0f) sum = fmaf(same, to_f32<T>(input[(size_t)token * input_stride + i]), sum);
+        out[at] = sum;
+    }
+}
+
+static int terms_fit(const FeedForwardTerms& f, int hidden) {
+    if (hidden <= 0 || (f.sorted && (f.top <= 0 || !f.slot_of || !f.weights))) return KIRAI_ERR_BAD_SIZE;
+    const bool reads_gates = f.same_count > 0 || (f.shared && f.share_col >= 0);
+    if (reads_gates && !f.gates) return KIRAI_ERR_BAD_SIZE;
+    if (f.same_count > 0 && (f.same_col < 0 || f.same_col + f.same_count > f.gates_stride)) return KIRAI_ERR_BAD_SIZE;
+    return f.shared && f.share_col >= f.gates_stride ? KIRAI_ERR_BAD_SIZE : 0;
+}
+
+// Refuses (KIRAI_ERR_UNSUPPORTED) what route_combine_norm_add refuses.
+KIRAI_EXPORT int kirai_terms_norm_add(float* resid, const float* routed, const void* sorted, const int* slot_of, const float* weights, int top,
+                                      const float* shared, int share_col, int same_col, int same_count, const float* gates, long gates_stride,
+                                      const float* norm_weight, void* copy, int tokens, int hidden, float eps, cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    const FeedForwardTerms f{routed, (const bf16*)sorted, slot_of, weights, shared, gates, gates_stride, top, share_col, same_col, same_count};
+    const int status = terms_fit(f, hidden);
+    if (status != 0) return status;
+    if (hidden % 4 != 0 || hidden > 4 * 4 * 512 ||
+        (((uintptr_t)resid | (uintptr_t)routed | (uintptr_t)sorted | (uintptr_t)shared | (uintptr_t)norm_weight | (uintptr_t)copy) & 15) != 0)
+        return KIRAI_ERR_UNSUPPORTED;
+    const int threads = hidden <= 4 * 4 * 128 ? 128 : (hidden <= 4 * 4 * 256 ? 256 : 512);
+    return launch_pdl(terms_norm_add_kernel<4>, dim3(tokens), dim3(threads), 0, stream, 1u, resid, f, norm_weight, (bf16*)copy, hidden, eps);
+}
+
+template <typename T>
+static int terms_sum_launch(const FeedForwardTerms& f, const void* input, long input_stride, float* out, int tokens, int hidden,
+                            cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    const int status = terms_fit(f, hidden);
+    if (status != 0) return status;
+    if (f.same_count > 0 && !input) return KIRAI_ERR_BAD_SIZE;
+    return launch_pdl(terms_sum_kernel<T>, dim3(tokens), dim3(hidden >= 2048 ? 256 : 128), 0, stream, 1u, f, (const T*)input, input_stride, out, hidden);
+}
+KIRAI_EXPORT int kirai_terms_sum_f32(const void* input, long input_stride, const float* routed, const void* sorted, const int* slot_of,
+                                      const float* weights, int top, const float* shared, int share_col, int same_col, int same_count,
+                                      const float* gates, long gates_stride, float* out, int tokens, int hidden, cudaStream_t stream) {
+    const FeedForwardTerms f{routed, (const bf16*)sorted, slot_of, weights, shared, gates, gates_stride, top, share_col, same_col, same_count};
+    return terms_sum_launch<float>(f, input, input_stride, out, tokens, hidden, stream);
+}
+KIRAI_EXPORT int kirai_terms_sum_bf16(const void* input, long input_stride, const float* routed, const void* sorted, const int* slot_of,
+                                      const float* weights, int top, const float* shared, int share_col, int same_col, int same_count,
+                                      const float* gates, long gates_stride, float* out, int tokens, int hidden, cudaStream_t stream) {
+    const FeedForwardTerms f{routed, (const bf16*)sorted, slot_of, weights, shared, gates, gates_stride, top, share_col, same_col, same_count};
+    return terms_sum_launch<bf16>(f, input, input_stride, out, tokens, hidden, stream);
 }

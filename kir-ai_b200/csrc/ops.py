@@ -303,6 +303,32 @@ def embedding_scaled(table: torch.Tensor, ids: torch.Tensor, scale: float, posit
     return out, copy
 
 
+def embedding_norm(table: torch.Tensor, ids: torch.Tensor, weight: torch.Tensor, eps: float, copy_dtype: Optional[torch.dtype] = None):
+    """Rows ``ids`` of the row-major ``table`` [V, H], each divided by its root mean square (``eps`` inside the root) and
+    multiplied by ``weight`` [H]: (the 32-bit stream [T, H], its bfloat16 copy when ``copy_dtype`` asks for it, else None)."""
+    _need_cuda(table, ids, weight)
+    assert ids.dtype == torch.int32 and ids.is_contiguous() and table.dim() == 2 and table.is_contiguous()
+    tokens, hidden = ids.numel(), table.shape[1]
+    assert weight.dtype == torch.float32 and weight.numel() == hidden and weight.is_contiguous()
+    out = torch.empty((tokens, hidden), dtype=torch.float32, device=table.device)
+    copy = torch.empty((tokens, hidden), dtype=torch.bfloat16, device=table.device) if copy_dtype == torch.bfloat16 else None
+    _call(f"kirai_embedding_norm_{_suffix(table.dtype)}", _ptr(table), _ptr(ids), _ptr(weight), _ptr(out), _ptr(copy), _i(tokens), _i(hidden),
+          _i(table.shape[0]), _f(eps), _ptr(error_flag(table.device)), _stream())
+    return out, copy
+
+
+def token_gate(z: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, first: int) -> torch.Tensor:
+    """gelu_tanh(``z`` [T, D], float32) times columns [first, first + D) of the rows ``ids`` of ``table`` [V, C]; [T, D] in the
+    table's dtype."""
+    _need_cuda(z, table, ids)
+    assert z.dtype == torch.float32 and z.dim() == 2 and z.is_contiguous() and table.dim() == 2 and table.is_contiguous()
+    assert ids.dtype == torch.int32 and ids.is_contiguous() and ids.numel() == z.shape[0] and first + z.shape[1] <= table.shape[1]
+    out = torch.empty(z.shape, dtype=table.dtype, device=z.device)
+    _call(f"kirai_token_gate_{_suffix(table.dtype)}", _ptr(z), _ptr(table), _ptr(ids), _ptr(out), _i(z.shape[0]), _i(z.shape[1]),
+          _l(table.shape[1]), _l(first), _i(table.shape[0]), _ptr(error_flag(z.device)), _stream())
+    return out
+
+
 def norm_add(resid: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float, copy_dtype: Optional[torch.dtype] = None):
     """The norm on a sub-layer's output: ``resid`` (32-bit, in place) += RMSNorm(``y``) with ``weight``; ``y`` [T, H] is
     32-bit.  Returns the new stream rounded to bfloat16 when ``copy_dtype`` asks for it (what the next sub-layer
@@ -688,17 +714,18 @@ def rms_pair_mean(a: torch.Tensor, b: torch.Tensor, weight_a: torch.Tensor, weig
 
 
 def gated_group_norm(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, groups: int, gate_first: bool,
-                     out_dtype: torch.dtype) -> torch.Tensor:
+                     out_dtype: torch.dtype, silu_after: bool = False) -> torch.Tensor:
     """``y`` [T, W] (float32; a run of columns of a wider tensor is allowed, as for ``gate``) through a gate and a
     unit-RMS norm over ``groups`` equal parts of a row (``eps`` inside the root), times ``weight`` [W].
-    ``gate_first``: (y * silu(gate)) is normed; else y is normed and then multiplied by sigmoid(gate)."""
+    ``gate_first``: (y * silu(gate)) is normed; else y is normed and then multiplied by sigmoid(gate), or with
+    ``silu_after`` by silu(gate)."""
     _need_cuda(y, gate, weight)
     assert y.dtype == gate.dtype == torch.float32 and y.dim() == 2 and y.shape == gate.shape and y.stride(1) == gate.stride(1) == 1
     width = y.shape[1]
     assert width % groups == 0 and weight.dtype == torch.float32 and weight.numel() == width and weight.is_contiguous()
     out = torch.empty((y.shape[0], width), dtype=out_dtype, device=y.device)
     _call(f"kirai_gated_group_norm_{_suffix(out_dtype)}", _ptr(y), _l(y.stride(0)), _ptr(gate), _l(gate.stride(0)), _ptr(weight),
-          _f(eps), _ptr(out), _i(y.shape[0]), _i(groups), _i(width // groups), _i(0 if gate_first else 1), _stream())
+          _f(eps), _ptr(out), _i(y.shape[0]), _i(groups), _i(width // groups), _i(0 if gate_first else (2 if silu_after else 1)), _stream())
     return out
 
 
@@ -935,6 +962,43 @@ def matrix_memory_walk(rows: torch.Tensor, in_bias: Optional[torch.Tensor], keep
     return o
 
 
+def channel_scan(rows: torch.Tensor, up: torch.Tensor, bias: torch.Tensor, tau: float, q_scale: float, state: torch.Tensor, batch,
+                 heads: int, key_dim: int, value_dim: int, norm: torch.Tensor, eps: float, out_dtype: torch.dtype,
+                 walk_limit: Optional[int] = None, chain_limit: Optional[int] = None) -> torch.Tensor:
+    """Gated linear attention over each request's tokens of this step.  ``rows`` [T, 2 H d + 2 H dv + r] (float32): q [H d],
+    k [H d], v [H dv], the output gate [H dv] and the short row u [r] of each token; ``up`` [r, H d] and ``bias`` [H d]
+    (float32): a = sigmoid(u up + bias)^(1 / tau) per key column.  Per head S <- diag(a) S + k v^T, o = S^T (q q_scale), S
+    [d, dv] in the request's slot of ``state`` [slots, L] (S [H, d, dv] from column 0).  Returns, in ``out_dtype``
+    [T, H dv], each head's o divided by its root mean square (``eps`` inside the root), times ``norm`` [H dv] (every head's
+    part the same) and silu(gate).  A step whose longest run of tokens is above ``walk_limit`` takes the runs a chunk of
+    tokens at a time, and above ``chain_limit`` the chunks side by side."""
+    _need_cuda(rows, up, bias, state, norm)
+    width, rank = heads * key_dim, up.shape[0]
+    assert rows.dtype == torch.float32 and rows.dim() == 2 and rows.stride(1) == 1 and rows.shape[1] == 2 * width + 2 * heads * value_dim + rank
+    assert up.dtype == bias.dtype == norm.dtype == torch.float32 and up.shape == (rank, width) and up.is_contiguous()
+    assert bias.numel() == width and bias.is_contiguous() and norm.numel() == heads * value_dim and norm.is_contiguous()
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous() and tau > 0.0
+    tokens = rows.shape[0]
+    common = (_ptr(rows), _l(rows.stride(0)), _ptr(up), _ptr(bias), _f(1.0 / tau), _f(q_scale), _ptr(state), _l(state.shape[1]),
+              _ptr(batch.query_start), _ptr(batch.slots))
+    sizes = (_i(batch.num_requests), _i(heads), _i(key_dim), _i(value_dim), _i(rank), _i(state.shape[0]))
+    fits = library().kirai_channel_chunks_fit
+    fits.restype = ctypes.c_int
+    if batch.max_query_len <= (STATE_WALK_LIMIT if walk_limit is None else walk_limit) or not fits(_i(key_dim), _i(rank)):
+        out = torch.empty((tokens, heads * value_dim), dtype=out_dtype, device=rows.device)
+        _call(f"kirai_channel_walk_{_suffix(out_dtype)}", *common, _ptr(norm), _f(eps), _ptr(out), *sizes, _i(batch.max_query_len), _stream())
+        return out
+    o = torch.empty((tokens, heads * value_dim), dtype=torch.float32, device=rows.device)
+    chunk = int(library().kirai_state_chunk_tokens())
+    units = tokens // chunk + batch.num_requests
+    tiles = torch.empty((units, heads, 2 * key_dim + chunk, chunk), dtype=torch.float32, device=rows.device)
+    kept = torch.empty((units, heads, key_dim), dtype=torch.float32, device=rows.device)
+    side = _state_side(batch, tokens, heads, key_dim, value_dim, False, rows.device, chain_limit)[1]
+    _call("kirai_channel_chunks", *common, _ptr(o), _ptr(tiles), _ptr(kept), _ptr(side), *sizes, _i(units), _stream())
+    gate = rows[:, 2 * width + heads * value_dim : 2 * width + 2 * heads * value_dim]
+    return gated_group_norm(o, gate, norm, eps, heads, False, out_dtype, silu_after=True)
+
+
 def head_gate_(x: torch.Tensor, gate: torch.Tensor, heads: int, used: int, pad_dim: int, out: Optional[torch.Tensor] = None,
                factor: float = 1.0) -> torch.Tensor:
     """``x`` [T, heads * pad_dim] (in place): the first ``used`` columns of head h times ``factor`` * sigmoid(gate[t, h]);
@@ -959,18 +1023,21 @@ def softcap_(x: torch.Tensor, cap: float) -> torch.Tensor:
 
 
 def gated_expert_gate(gate_up: torch.Tensor, gates: torch.Tensor, ff: int, activation: str = "silu", limit: float = 0.0,
-                      slope: float = 1.0, interleaved: bool = False) -> torch.Tensor:
+                      slope: float = 1.0, interleaved: bool = False, experts: Optional[int] = None, shared_ff: int = 0,
+                      shared_col: int = 0) -> torch.Tensor:
     """Stacked gated experts: ``gate_up`` [T, experts * 2 ff] (per expert ff gate columns, then ff up columns) becomes
-    [T, experts * ff] = act(gate) * up * gates[t, expert] (``gates`` float32 [T, experts], zero where not chosen);
+    [T, experts * ff] = act(gate) * up * gates[t, expert] (``gates`` float32 [T, >= experts], zero where not chosen;
+    ``experts`` None: as many as it has columns);
     the activations are those of ``gated_activation``.  ``interleaved``: an expert's columns come as 8 gate columns,
-    their 8 up columns, 8 gate columns, ... (see ``interleave_gate_up``)."""
+    their 8 up columns, 8 gate columns, ... (see ``interleave_gate_up``).  ``shared_ff`` S: behind the experts stands one
+    branch of S hidden columns (2 S columns of ``gate_up`` in the same order within), weighted by gates[t, shared_col]."""
     _need_cuda(gate_up, gates)
     assert gate_up.dim() == 2 and gate_up.is_contiguous() and gates.dtype == torch.float32 and gates.is_contiguous()
-    experts = gates.shape[1]
-    assert gate_up.shape == (gates.shape[0], experts * 2 * ff)
-    out = torch.empty((gate_up.shape[0], experts * ff), dtype=gate_up.dtype, device=gate_up.device)
-    _call(f"kirai_gated_expert_gate_{_suffix(gate_up.dtype)}", _ptr(gate_up), _ptr(gates), _ptr(out), _i(gate_up.shape[0]),
-          _i(experts), _i(ff), _i(GATED_ACTIVATIONS[activation]), _f(limit), _f(slope), _i(int(interleaved)), _stream())
+    experts = gates.shape[1] if experts is None else experts
+    assert gate_up.shape == (gates.shape[0], 2 * (experts * ff + shared_ff))
+    out = torch.empty((gate_up.shape[0], experts * ff + shared_ff), dtype=gate_up.dtype, device=gate_up.device)
+    _call(f"kirai_gated_expert_gate_{_suffix(gate_up.dtype)}", _ptr(gate_up), _ptr(gates), _l(gates.shape[1]), _ptr(out), _i(gate_up.shape[0]),
+          _i(experts), _i(ff), _i(shared_ff), _i(shared_col), _i(GATED_ACTIVATIONS[activation]), _f(limit), _f(slope), _i(int(interleaved)), _stream())
     return out
 
 
@@ -993,18 +1060,23 @@ def _router_arrivals(device: torch.device, tokens: int) -> torch.Tensor:
 
 
 def _router_rule(over_all: bool, rule: Optional[dict], experts: int, device):
-    """The kernels' arguments for how weights come from logits: (mode, correction, groups, keep).  ``rule`` is None
-    (softmax over the chosen logits, or over all with ``over_all``) or a dict with ``correction`` (a tensor [experts],
-    float32, or None), ``groups`` and ``keep``: sigmoid scores, the choice by score + correction among the ``keep``
-    best of ``groups`` equal groups of neighbouring experts (a group's mark is the sum of its two largest choice
-    scores), the weights the chosen scores as they are."""
+    """The kernels' arguments for how weights come from logits: (mode, correction, groups, keep, scale, extra).  ``rule`` is
+    None (softmax over the chosen logits, or over all with ``over_all``) or a dict with ``correction`` (a tensor [experts],
+    float32, or None) and
+    * ``groups`` and ``keep``: sigmoid scores, the choice by score + correction among the ``keep``
+      best of ``groups`` equal groups of neighbouring experts (a group's mark is the sum of its two largest choice
+      scores), the weights the chosen scores as they are; or
+    * ``scale``: softmax scores over all experts, the choice by score + correction, the weights the chosen scores divided by
+      their sum (+ 1e-20), times ``scale``; ``extra`` columns behind the experts' become sigmoids of their logits."""
     if rule is None:
-        return _i(int(over_all)), _ptr(None), _i(1), _i(1)
+        return _i(int(over_all)), _ptr(None), _i(1), _i(1), _f(1.0), _i(0)
     correction = rule.get("correction")
     if correction is not None:
         _need_cuda(correction)
         assert correction.dtype == torch.float32 and correction.numel() == experts and correction.is_contiguous()
-    return _i(2), _ptr(correction), _i(int(rule.get("groups", 1))), _i(int(rule.get("keep", 1)))
+    mode = 3 if rule.get("scale") is not None else 2
+    return (_i(mode), _ptr(correction), _i(int(rule.get("groups", 1))), _i(int(rule.get("keep", 1))),
+            _f(float(rule.get("scale") or 1.0)), _i(int(rule.get("extra", 0))))
 
 
 def router_gates(x: torch.Tensor, router: torch.Tensor, top: int, want_chosen: bool = False, over_all: bool = False,
@@ -1013,12 +1085,15 @@ def router_gates(x: torch.Tensor, router: torch.Tensor, top: int, want_chosen: b
     largest chosen (the lower index on a tie), softmax over the chosen logits alone.  Returns gates [T, experts]
     (float32, zero where not chosen); with ``want_chosen`` also (ids [T, top] int32, weights [T, top] float32) in the
     order of choice.  ``over_all``: the weights are the chosen experts' shares of the softmax over ALL logits instead
-    (they then do not sum to one).  ``rule``: sigmoid scores with a correction and groups, see ``_router_rule``."""
+    (they then do not sum to one).  ``rule``: scores with a correction, and further rows of ``router`` behind the experts'
+    whose logits come out as sigmoids in columns behind theirs, see ``_router_rule``."""
     _need_cuda(x, router)
+    columns = router.shape[0]
+    experts = columns - (int(rule.get("extra", 0)) if rule else 0)
     assert x.dim() == 2 and x.stride(1) == 1 and router.dtype == torch.float32 and router.is_contiguous()
-    assert router.shape[1] == x.shape[1] and 0 < top <= router.shape[0]
-    tokens, experts = x.shape[0], router.shape[0]
-    gates = torch.empty((tokens, experts), dtype=torch.float32, device=x.device)
+    assert router.shape[1] == x.shape[1] and 0 < top <= experts
+    tokens = x.shape[0]
+    gates = torch.empty((tokens, columns), dtype=torch.float32, device=x.device)
     ids = torch.empty((tokens, top), dtype=torch.int32, device=x.device) if want_chosen else None
     weights = torch.empty((tokens, top), dtype=torch.float32, device=x.device) if want_chosen else None
     _call(f"kirai_router_gates_{_suffix(x.dtype)}", _ptr(x), _l(x.stride(0)), _ptr(router), _ptr(gates), _ptr(ids), _ptr(weights),
@@ -1031,8 +1106,9 @@ def router_choose_(logits: torch.Tensor, top: int, want_chosen: bool = False, ov
     """The choice alone: ``logits`` [T, experts] (float32, as a product left them) become the routing weights in place
     (see ``router_gates``).  Returns what ``router_gates`` returns."""
     _need_cuda(logits)
-    assert logits.dtype == torch.float32 and logits.dim() == 2 and logits.is_contiguous() and 0 < top <= logits.shape[1]
-    tokens, experts = logits.shape
+    experts = logits.shape[1] - (int(rule.get("extra", 0)) if rule else 0)
+    assert logits.dtype == torch.float32 and logits.dim() == 2 and logits.is_contiguous() and 0 < top <= experts
+    tokens = logits.shape[0]
     ids = torch.empty((tokens, top), dtype=torch.int32, device=logits.device) if want_chosen else None
     weights = torch.empty((tokens, top), dtype=torch.float32, device=logits.device) if want_chosen else None
     _call("kirai_router_choose", _ptr(logits), _ptr(ids), _ptr(weights), _i(tokens), _i(experts), _i(top),
@@ -1113,6 +1189,54 @@ def route_combine_norm_add(resid: torch.Tensor, y: torch.Tensor, slot_of: torch.
     _call("kirai_route_combine_norm_add_bf16", _ptr(resid), _ptr(y), _ptr(slot_of), _ptr(weights), _ptr(norm_weight), _ptr(copy),
           _i(resid.shape[0]), _i(resid.shape[1]), _i(slot_of.shape[1]), _f(eps), _stream())
     return copy
+
+
+def _terms_args(hidden: int, tokens: int, routed, sorted_rows, shared, gates, share_col: int, same: tuple):
+    """The kernels' arguments for the terms of a feed-forward (see ``terms_norm_add``)."""
+    y, slot_of, weights = sorted_rows if sorted_rows is not None else (None, None, None)
+    _need_cuda(routed, y, slot_of, weights, shared, gates)
+    for t in (routed, shared):
+        assert t is None or (t.dtype == torch.float32 and t.shape == (tokens, hidden) and t.is_contiguous())
+    top = 0
+    if y is not None:
+        assert y.dtype == torch.bfloat16 and y.dim() == 2 and y.is_contiguous() and y.shape[1] == hidden
+        assert slot_of.dtype == torch.int32 and slot_of.is_contiguous() and slot_of.shape[0] == tokens
+        assert weights.dtype == torch.float32 and weights.shape == slot_of.shape and weights.is_contiguous()
+        top = slot_of.shape[1]
+    if gates is not None:
+        assert gates.dtype == torch.float32 and gates.dim() == 2 and gates.shape[0] == tokens and gates.is_contiguous()
+    return (_ptr(routed), _ptr(y), _ptr(slot_of), _ptr(weights), _i(top), _ptr(shared), _i(share_col), _i(same[0]), _i(same[1]), _ptr(gates),
+            _l(gates.shape[1] if gates is not None else 0))
+
+
+def terms_norm_add(resid: torch.Tensor, routed: Optional[torch.Tensor], sorted_rows: Optional[tuple], shared: Optional[torch.Tensor],
+                   gates: Optional[torch.Tensor], share_col: int, same: tuple, norm_weight: torch.Tensor, eps: float,
+                   copy_dtype: Optional[torch.dtype] = None):
+    """A feed-forward's terms summed, normed and added in one pass: y = ``routed`` [T, H] (float32, or None) + the rows sorted
+    by expert, ``sorted_rows`` = (rows, slot_of, weights) as for ``route_combine``, or None, + gates[t, share_col] *
+    ``shared`` [T, H] (float32, or None; ``share_col`` < 0: times one) + (the sum of ``same`` = (first, count) columns of
+    ``gates``) * the stream itself; ``resid`` (32-bit, in place) += RMSNorm(y) with ``norm_weight``.  Returns the stream's
+    bfloat16 copy when ``copy_dtype`` asks for it.  Widths as for ``route_combine_norm_add``."""
+    _need_cuda(resid, norm_weight)
+    assert resid.dtype == torch.float32 and resid.dim() == 2 and resid.is_contiguous()
+    tokens, hidden = resid.shape
+    assert norm_weight.dtype == torch.float32 and norm_weight.numel() == hidden and norm_weight.is_contiguous()
+    copy = torch.empty(resid.shape, dtype=torch.bfloat16, device=resid.device) if copy_dtype == torch.bfloat16 else None
+    _call("kirai_terms_norm_add", _ptr(resid), *_terms_args(hidden, tokens, routed, sorted_rows, shared, gates, share_col, same),
+          _ptr(norm_weight), _ptr(copy), _i(tokens), _i(hidden), _f(eps), _stream())
+    return copy
+
+
+def terms_sum(x: torch.Tensor, routed: Optional[torch.Tensor], sorted_rows: Optional[tuple], shared: Optional[torch.Tensor],
+              gates: Optional[torch.Tensor], share_col: int, same: tuple) -> torch.Tensor:
+    """The sum of ``terms_norm_add`` alone, [T, H] (float32), with the experts' input ``x`` [T, H] in place of the stream."""
+    _need_cuda(x)
+    assert x.dim() == 2 and x.stride(1) == 1
+    tokens, hidden = x.shape
+    out = torch.empty((tokens, hidden), dtype=torch.float32, device=x.device)
+    _call(f"kirai_terms_sum_{_suffix(x.dtype)}", _ptr(x), _l(x.stride(0)),
+          *_terms_args(hidden, tokens, routed, sorted_rows, shared, gates, share_col, same), _ptr(out), _i(tokens), _i(hidden), _stream())
+    return out
 
 
 def linear_grouped(x: torch.Tensor, weight, groups: int, tile_group: torch.Tensor, out_dtype: torch.dtype = torch.bfloat16,

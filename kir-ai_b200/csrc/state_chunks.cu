@@ -18,14 +18,11 @@
 // matrix products over shared tiles, a thread holding a 4 x 4 tile of each.  Gates, decays, scores, sums and the
 // state are 32-bit.  The matrix memory's new normaliser and maximum go to a side buffer and from there to the slot in
 // a second kernel, since every block of a head reads the old ones.
+#include "chunk_tiles.cuh"
 #include "common.cuh"
 #include "state_math.cuh"
 
 namespace {
-
-constexpr int CHUNK = 64;         // tokens a chunk
-constexpr int PITCH = CHUNK + 4;  // floats a row of the tiles that keep a chunk's tokens along a row
-constexpr int THREADS = 256;      // 16 x 16 threads, 4 x 4 entries each
 
 struct ChunkScan {
     const float* q;  // [*, groups d] (row stride q_stride): what reads the state
@@ -48,39 +45,6 @@ struct ChunkScan {
     float* out;  // [*, heads dv]
     int heads, groups, d, dv, cols, num_slots, memory;
 };
-
-__host__ __device__ inline int cols_pitch(int cols) { return (cols + 15) / 16 * 16; }
-
-// A 4-byte copy from global to shared memory that the thread does not wait for (any address, any stride).
-__device__ __forceinline__ void copy_async(float* to, const float* from) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((unsigned)__cvta_generic_to_shared(to)), "l"(from) : "memory");
-}
-__device__ __forceinline__ void copies_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
-
-// `len` rows of `d` columns from `from` (row stride `stride`) into a tile that keeps tokens along a row, [d][PITCH];
-// the columns of tokens that the chunk does not have are zero.
-__device__ __forceinline__ void fetch_across(float* tile, const float* from, long stride, int len, int d) {
-    const int lane = threadIdx.x & 31;
-    for (int t = threadIdx.x >> 5; t < CHUNK; t += THREADS / 32) {  // a warp takes a token's row
-        const float* row = from + t * stride;
-        if (t < len)
-            for (int kd = lane; kd < d; kd += 32) copy_async(tile + kd * PITCH + t, row + kd);
-        else
-            for (int kd = lane; kd < d; kd += 32) tile[kd * PITCH + t] = 0.0f;
-    }
-}
-
-// `len` rows of `cols` columns into a tile [CHUNK][cp]; zero elsewhere.
-__device__ __forceinline__ void fetch_along(float* tile, const float* from, long stride, int len, int cols, int cp) {
-    const int c = threadIdx.x & 15;
-    for (int t = threadIdx.x >> 4; t < CHUNK; t += THREADS / 16) {
-        const float* row = from + t * stride;
-        for (int at = c; at < cp; at += 16) {
-            if (t < len && at < cols) copy_async(tile + t * cp + at, row + at);
-            else tile[t * cp + at] = 0.0f;
-        }
-    }
-}
 
 __host__ __device__ inline long chunk_scan_floats(int d, int cols) {
     const int cp = cols_pitch(cols);
@@ -376,27 +340,6 @@ __global__ void __launch_bounds__(THREADS) chunk_scan_kernel(const ChunkScan a) 
 //      chunk's START where U was and moves on by S <- exp(M - Xf) S + exp(X'_last - Xf) U, Xf = max(M, X'_last),
 //      M <- G_last + Xf (the state space has M = 0 throughout and X'_last = -G_last, so S <- exp(G_last) S + U);
 //   3. chunk_out: block (chunk, head, run of columns) reads the chunk's tokens out of the state at its start.
-// The step's chunks are numbered request by request; a block finds its request by a walk over the row boundaries.
-struct ChunkPlace {
-    int request, chunk, chunks, len;
-    long row0;
-};
-
-__device__ __forceinline__ bool find_chunk(const int* __restrict__ query_start, int requests, int at, ChunkPlace& place) {
-    for (int r = 0; r < requests; ++r) {
-        const int first = query_start[r], count = query_start[r + 1] - first;
-        const int chunks = (count + CHUNK - 1) / CHUNK;
-        if (at < chunks) {
-            place.request = r, place.chunk = at, place.chunks = chunks;
-            place.len = min(CHUNK, count - at * CHUNK);
-            place.row0 = (long)first + (long)at * CHUNK;
-            return true;
-        }
-        at -= chunks;
-    }
-    return false;
-}
-
 struct ChunkSide {
     float* U;      // [chunks of the step, heads, d, dv]: a chunk's own share, then the state at its start
     float* u;      // [chunks, heads, d]: likewise for the normaliser (matrix memory)
@@ -444,8 +387,7 @@ __global__ void __launch_bounds__(256) chunk_carry_kernel(const ChunkScan a, con
     const int request = blockIdx.x, head = blockIdx.y;
     const long entry = blockIdx.z * 256L + threadIdx.x;
     const long cells = (long)a.d * a.dv;
-    int before = 0;
-    for (int r = 0; r < request; ++r) before += (a.query_start[r + 1] - a.query_start[r] + CHUNK - 1) / CHUNK;
+    const int before = first_chunk(a.query_start, request);
     const int chunks = (a.query_start[request + 1] - a.query_start[request] + CHUNK - 1) / CHUNK;
     const int slot = a.slots[request];
     pdl_wait();
@@ -548,16 +490,6 @@ int choose_cols(int requests, int heads, int d, int dv, bool side_by_side, long*
     *bytes = chunk_scan_floats(d, cols) * 4;
     return *bytes <= limit ? cols : 0;
 }
-
-template <typename Kernel>
-int grant_shared(Kernel kernel, long bytes, long* granted) {
-    if (bytes <= *granted) return 0;
-    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess) return launch_status();
-    *granted = bytes;
-    return 0;
-}
-
-#define KIRAI_BY_RUNS(runs, name) ((runs) == 1 ? name<1> : (runs) == 2 ? name<2> : (runs) == 3 ? name<3> : name<4>)
 
 // `units` > 0: the chunks side by side, with `side`'s buffers for `units` chunks (at least tokens / 64 + requests).
 int chunk_scan_launch(ChunkScan a, int requests, int units, ChunkSide side, cudaStream_t stream) {

@@ -112,7 +112,8 @@ KIRAI_EXPORT int kirai_rms_pair_mean(const float* a, const float* b, const float
 // ------------------------------------------------------- gate and unit-RMS norm over groups
 // A warp per (row, group), or a block where a group is wide.  y [T, width] (float32, row stride y_stride), gate
 // (float32, row stride g_stride), weight [width].  mode 0: v = y * silu(gate), out = v / rms_group(v) * weight (the gate
-// comes before the norm); mode 1: out = y / rms_group(y) * weight * sigmoid(gate) (the gate comes after it).
+// comes before the norm); mode 1: out = y / rms_group(y) * weight * sigmoid(gate) (the gate comes after it); mode 2: the
+// same as mode 1 with silu(gate).
 template <typename O, int WARPS>
 __global__ void gated_group_norm_kernel(const float* __restrict__ y, long y_stride, const float* __restrict__ gate, long g_stride,
                                         const float* __restrict__ weight, float eps, O* __restrict__ out, long rows, int groups,
@@ -139,7 +140,7 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, long y_stri
     const float r = rsqrtf(sum / (float)group_width + eps);
     O* po = out + row * (long)groups * group_width + c0;
     for (int c = lane; c < group_width; c += step) {
-        const float v = mode == 0 ? py[c] * sf_silu(pg[c]) : py[c] * sf_sigmoid(pg[c]);
+        const float v = mode == 1 ? py[c] * sf_sigmoid(pg[c]) : py[c] * sf_silu(pg[c]);
         po[c] = from_f32<O>(v * r * weight[c0 + c]);
     }
 }
@@ -172,7 +173,8 @@ __global__ void __launch_bounds__(1024) gated_group_norm_vec_kernel(const float*
         if (c >= group_width) break;
         if (mode == 0) v[n].x *= sf_silu(g[n].x), v[n].y *= sf_silu(g[n].y), v[n].z *= sf_silu(g[n].z), v[n].w *= sf_silu(g[n].w);
         sum += (v[n].x * v[n].x + v[n].y * v[n].y) + (v[n].z * v[n].z + v[n].w * v[n].w);
-        if (mode != 0) v[n].x *= sf_sigmoid(g[n].x), v[n].y *= sf_sigmoid(g[n].y), v[n].z *= sf_sigmoid(g[n].z), v[n].w *= sf_sigmoid(g[n].w);
+        if (mode == 1) v[n].x *= sf_sigmoid(g[n].x), v[n].y *= sf_sigmoid(g[n].y), v[n].z *= sf_sigmoid(g[n].z), v[n].w *= sf_sigmoid(g[n].w);
+        if (mode == 2) v[n].x *= sf_silu(g[n].x), v[n].y *= sf_silu(g[n].y), v[n].z *= sf_silu(g[n].z), v[n].w *= sf_silu(g[n].w);
     }
     sum = block_sum(sum, scratch);
     const float r = rsqrtf(sum / (float)group_width + eps);
@@ -199,7 +201,7 @@ template <typename O>
 static int gated_group_norm_launch(const float* y, long y_stride, const float* gate, long g_stride, const float* weight, float eps,
                                    void* out, int rows, int groups, int group_width, int mode, cudaStream_t stream) {
     if (rows <= 0) return 0;
-    if (groups <= 0 || group_width <= 0 || mode < 0 || mode > 1) return KIRAI_ERR_BAD_SIZE;
+    if (groups <= 0 || group_width <= 0 || mode < 0 || mode > 2) return KIRAI_ERR_BAD_SIZE;
     const long units = (long)rows * groups;
     const bool vec = group_width % 4 == 0 && group_width >= 512 && group_width <= 4 * 4 * 1024 && y_stride % 4 == 0 && g_stride % 4 == 0 &&
                      (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
@@ -559,22 +561,27 @@ KIRAI_EXPORT int kirai_softcap_rows(float* x, float cap, long total, cudaStream_
 // act 0: silu, 1: the tanh form of gelu, 2: the clamped form (clamped_gated_f32 with `limit` and `slope`).
 // `interleaved`: an expert's columns come as 8 gate columns, their 8 up columns, 8 gate columns, ... (the order in which
 // the tensor-core product's gated epilogue wants the matrices' rows; ff a multiple of 8).
+// `gates` has `gates_stride` numbers a row.  A branch of another size that every token runs may stand behind the experts:
+// its gate and up columns follow theirs (in the same order within), `shared_ff` hidden columns, weighted by number
+// `shared_col` of the token's row.
 template <typename T>
-__global__ void gated_expert_gate_kernel(const T* __restrict__ gate_up, const float* __restrict__ gates, T* __restrict__ out,
-                                         long rows, int experts, int ff, int act, float limit, float slope, int interleaved) {
+__global__ void gated_expert_gate_kernel(const T* __restrict__ gate_up, const float* __restrict__ gates, long gates_stride, T* __restrict__ out,
+                                         long rows, int experts, int ff, int shared_ff, int shared_col, int act, float limit, float slope,
+                                         int interleaved) {
     pdl_launch_dependents();
     pdl_wait();
-    const long per_row = (long)experts * ff, total = rows * per_row;
+    const long routed = (long)experts * ff, per_row = routed + shared_ff, total = rows * per_row;
     for (long at = blockIdx.x * (long)blockDim.x + threadIdx.x; at < total; at += (long)gridDim.x * blockDim.x) {
         const long row = at / per_row;
         const int col = (int)(at - row * per_row);
-        const int e = col / ff, j = col - e * ff;
-        const float weight = gates[row * experts + e];
+        const bool shared = col >= routed;
+        const int e = shared ? experts : col / ff, j = col - e * ff, size = shared ? shared_ff : ff;
+        const float weight = gates[row * gates_stride + (shared ? shared_col : e)];
         float value = 0.0f;
         if (weight != 0.0f) {
             const T* src = gate_up + row * 2 * per_row + (long)e * 2 * ff;
             const int at_gate = interleaved ? ((j >> 3) << 4) + (j & 7) : j;
-            const float g = to_f32<T>(src[at_gate]), u = to_f32<T>(src[interleaved ? at_gate + 8 : ff + j]);
+            const float g = to_f32<T>(src[at_gate]), u = to_f32<T>(src[interleaved ? at_gate + 8 : size + j]);
             value = act == 2 ? clamped_gated_f32(g, u, limit, slope) * weight : (act == 1 ? sf_gelu_tanh(g) : sf_silu(g)) * u * weight;
         }
         out[at] = from_f32<T>(value);
@@ -582,22 +589,27 @@ __global__ void gated_expert_gate_kernel(const T* __restrict__ gate_up, const fl
 }
 
 template <typename T>
-static int gated_expert_gate_launch(const void* gate_up, const float* gates, void* out, int rows, int experts, int ff, int act,
-                                    float limit, float slope, int interleaved, cudaStream_t stream) {
+static int gated_expert_gate_launch(const void* gate_up, const float* gates, long gates_stride, void* out, int rows, int experts, int ff,
+                                    int shared_ff, int shared_col, int act, float limit, float slope, int interleaved, cudaStream_t stream) {
     if (rows <= 0) return 0;
-    if (experts <= 0 || ff <= 0 || act < 0 || act > 2 || (act == 2 && !(limit > 0.0f)) || (interleaved && ff % 8 != 0))
+    if (experts <= 0 || ff <= 0 || act < 0 || act > 2 || (act == 2 && !(limit > 0.0f)) || (interleaved && (ff % 8 != 0 || shared_ff % 8 != 0)))
         return KIRAI_ERR_BAD_SIZE;
-    const long total = (long)rows * experts * ff;
+    if (shared_ff < 0 || gates_stride < experts || (shared_ff > 0 && (shared_col < 0 || shared_col >= gates_stride))) return KIRAI_ERR_BAD_SIZE;
+    const long total = (long)rows * ((long)experts * ff + shared_ff);
     const unsigned blocks = (unsigned)min((total + 255) / 256, (long)148 * 16);
-    return launch_pdl(gated_expert_gate_kernel<T>, dim3(blocks), dim3(256), 0, stream, 1u, (const T*)gate_up, gates, (T*)out,
-                      (long)rows, experts, ff, act, limit, slope, interleaved);
+    return launch_pdl(gated_expert_gate_kernel<T>, dim3(blocks), dim3(256), 0, stream, 1u, (const T*)gate_up, gates, gates_stride, (T*)out,
+                      (long)rows, experts, ff, shared_ff, shared_col, act, limit, slope, interleaved);
 }
 
-KIRAI_EXPORT int kirai_gated_expert_gate_f32(const void* gate_up, const float* gates, void* out, int rows, int experts, int ff,
-                                             int act, float limit, float slope, int interleaved, cudaStream_t stream) {
-    return gated_expert_gate_launch<float>(gate_up, gates, out, rows, experts, ff, act, limit, slope, interleaved, stream);
+KIRAI_EXPORT int kirai_gated_expert_gate_f32(const void* gate_up, const float* gates, long gates_stride, void* out, int rows, int experts,
+                                              int ff, int shared_ff, int shared_col, int act, float limit, float slope, int interleaved,
+                                              cudaStream_t stream) {
+    return gated_expert_gate_launch<float>(gate_up, gates, gates_stride, out, rows, experts, ff, shared_ff, shared_col, act, limit, slope,
+                                         interleaved, stream);
 }
-KIRAI_EXPORT int kirai_gated_expert_gate_bf16(const void* gate_up, const float* gates, void* out, int rows, int experts, int ff,
-                                              int act, float limit, float slope, int interleaved, cudaStream_t stream) {
-    return gated_expert_gate_launch<bf16>(gate_up, gates, out, rows, experts, ff, act, limit, slope, interleaved, stream);
+KIRAI_EXPORT int kirai_gated_expert_gate_bf16(const void* gate_up, const float* gates, long gates_stride, void* out, int rows, int experts,
+                                              int ff, int shared_ff, int shared_col, int act, float limit, float slope, int interleaved,
+                                              cudaStream_t stream) {
+    return gated_expert_gate_launch<bf16>(gate_up, gates, gates_stride, out, rows, experts, ff, shared_ff, shared_col, act, limit, slope,
+                                         interleaved, stream);
 }
