@@ -2,6 +2,7 @@
 from .attention import GQAttention
 from .base import (FeedForward, KVCacheNeed, Mixer, Norm, Part, PositionEncoding, Runtime, StateNeed, StreamCopy, WeightSpec)
 from .block import Block
+from .decayed_attention import DecayedLinearAttention
 from .embedding import Embedding, OutputHead
 from .experts import RoutedExperts
 from .latent import LatentAttention
@@ -18,9 +19,11 @@ from .side_by_side import ScaledPairMixer, SideBySideMixer
 from .state_space import StateSpaceMixer
 from .streams import StreamConnection
 from .swiglu import GatedMLP, SwiGLU
+from .token_side import TokenSideInput
 from .two_map import TwoMapAttention
 
 __all__ = ["GQAttention", "FeedForward", "KVCacheNeed", "Mixer", "Norm", "Part", "PositionEncoding", "Runtime",
            "StateNeed", "StreamCopy", "WeightSpec", "RoutedExperts", "Block", "Embedding", "OutputHead", "Linear", "RMSNorm", "RotaryEmbedding", "SwiGLU",
            "GatedMLP", "LatentAttention", "LayerNorm", "MinGRU", "TokenShift", "DynamicTanh", "MatrixMemory", "SideBySideMixer",
-           "StateSpaceMixer", "StreamMerge", "PlainMLP", "GatedLinearRecurrence", "ScaledPairMixer", "StreamConnection", "TwoMapAttention"]
+           "StateSpaceMixer", "StreamMerge", "PlainMLP", "GatedLinearRecurrence", "ScaledPairMixer", "StreamConnection", "TwoMapAttention",
+           "DecayedLinearAttention", "TokenSideInput"]

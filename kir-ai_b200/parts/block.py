@@ -10,7 +10,8 @@ norms what a sub-layer produced, not what it reads: h' = h + norm1(mixer(h));
 out = h' + norm2(ffn(h')), the sub-layers reading the stream itself (rounded to
 the runtime dtype); such a block may have no feed-forward (``ffn`` and ``norm2``
 None), and it asks its sub-layers for 32-bit outputs (``out_dtype``), which the
-norm kernel reads.
+norm kernel reads.  An ``out_norm`` block may end with a ``side`` input (``parts.token_side.TokenSideInput``): something
+that is added into the stream from what the stream is by then and the token itself.
 
 Where the parts on both sides offer it, a norm is not a kernel of its own: the product before it adds into the
 stream and writes the norm's rows without their 1 / rms factor (``forward_into_norm``), and the product after it
@@ -61,7 +62,11 @@ def _offers(part, method: str, rows: int) -> bool:
 class Block(Part):
     def __init__(self, norm1: Norm, mixer: Mixer, norm2: Optional[Norm], ffn: Optional[FeedForward], arrangement: str = "pre_norm",
                  shift: Optional[Part] = None, residual_scale: Optional[float] = None, post_norm1: Optional[Norm] = None,
-                 post_norm2: Optional[Norm] = None, connection1: Optional[Part] = None, connection2: Optional[Part] = None):
+                 post_norm2: Optional[Norm] = None, connection1: Optional[Part] = None, connection2: Optional[Part] = None,
+                 side: Optional[Part] = None):
+        if side is not None and arrangement != "out_norm":
+            raise ValueError("an input of the token's own is built for the out_norm arrangement only")
+        self.side = side
         if (arrangement == "streams") != (connection1 is not None) or (connection2 is not None) != (arrangement == "streams" and ffn is not None):
             raise ValueError("the streams arrangement, and it alone, has a connection around every sub-layer")
         if arrangement == "streams" and ((ffn is None) != (norm2 is None) or shift is not None):
@@ -95,7 +100,7 @@ class Block(Part):
 
     def _parts(self):
         return [p for p in (self.norm1, self.connection1, self.shift, self.mixer, self.post_norm1, self.norm2, self.connection2, self.ffn,
-                            self.post_norm2) if p is not None]
+                            self.post_norm2, self.side) if p is not None]
 
     def shift_need(self):
         """What the block's token shift keeps per request (None without one)."""
@@ -265,4 +270,6 @@ class Block(Part):
                 x = self.ffn.forward_add_normed(x, batch, resid, spec)
             else:
                 x = self.norm2.add_normed(resid, self.ffn.forward(x if narrow else resid, batch))
+        if self.side is not None:
+            x = self.side.add(x if narrow else resid, resid, batch)
         return resid, StreamCopy(x if narrow else None)

@@ -23,6 +23,12 @@ gate in the same kernel) and W_o reads heads * value_dim columns as stored; the 
 projection.  A rotation that pairs neighbouring columns (``RotaryEmbedding(pairing="neighbours")``) has the rows that
 make the rotated query columns and the shared key part put in its ``head_order`` at load; a rotation with an
 ``amplitude`` is applied with it by both preparation kernels.
+
+``q_rank`` None: there is no query latent, queries are W_q h.  W_uk is then folded into W_q (rows W_uk,i^T W_q,i), and the
+folded queries, the latent's and the shared key part's rows and the gate's are one stacked product on h.  ``head_gate``
+(the name of a matrix [heads, hidden], in place of ``gate``): head i's values are multiplied by sigmoid(head_gate h)_i.  One
+number a head commutes with W_uv, so both folds stay and the sums of latents are multiplied.  ``sink`` (the name of a vector
+[heads]): every head's softmax has one more term exp(sink_i) in its denominator that no key or value stands behind.
 """
 from __future__ import annotations
 
@@ -38,12 +44,20 @@ from .rope import RotaryEmbedding
 class LatentAttention(Mixer):
     kernels_only = True
 
-    def __init__(self, prefix: str, hidden_size: int, heads: int, dim: int, rot_dim: int, value_dim: int, q_rank: int,
+    def __init__(self, prefix: str, hidden_size: int, heads: int, dim: int, rot_dim: int, value_dim: int, q_rank: Optional[int],
                  kv_rank: int, scale: float, eps: float, rotary: RotaryEmbedding, names: Optional[Dict[str, str]] = None,
-                 out_dtype: Optional[torch.dtype] = None, gate: Optional[str] = None):
-        n = {"dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "o": "o"}
+                 out_dtype: Optional[torch.dtype] = None, gate: Optional[str] = None,
+                 head_gate: Optional[str] = None, sink: Optional[str] = None):
+        n = {"q": "q", "dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "o": "o"}
         n.update(names or {})
         self.gate_name = prefix + gate if gate else None
+        self.head_gate_name = prefix + head_gate if head_gate else None
+        self.sink_name, self.sinks = prefix + sink if sink else None, None
+        self.direct = q_rank is None
+        if gate and (head_gate or self.direct):
+            raise ValueError("a gate per column goes with a query latent and no gate per head")
+        if head_gate and not self.direct:
+            raise ValueError("a gate per head is built for queries without a latent")
         if rotary.head_dim != rot_dim or rotary.rotary_dim != rot_dim or rotary.offset != 0:
             raise ValueError("the rotation of latent attention covers the whole shared key part")
         self.hidden_size, self.heads, self.dim, self.rot_dim, self.value_dim = hidden_size, heads, dim, rot_dim, value_dim
@@ -52,6 +66,14 @@ class LatentAttention(Mixer):
         self.pad_dim = -(-self.row // 8) * 8
         self.names = {key: prefix + value for key, value in n.items()}
         self.order = rotary.head_order()  # of the rotated columns, where the rotation pairs neighbours
+        if self.direct:
+            self.out = Linear([("", hidden_size)], heads * self.pad_dim)     # filled from o and uv at load
+            # [folded queries, latent, shared key part, gates], filled at load; zero rows behind them keep 16-byte rows
+            self.stack = -(-(heads * self.row + self.row + (heads if head_gate else 0)) // 4) * 4
+            self.down = Linear([("", self.stack)], hidden_size)
+            self.up_v = self.up_v_padded = None
+            self.q_norm = self.kv_norm = None
+            return
         sources = [(self.names["dq"], q_rank), (self.names["dkv"], kv_rank + rot_dim)]
         if self.gate_name:
             sources.append((self.gate_name, heads * value_dim))
@@ -78,7 +100,14 @@ class LatentAttention(Mixer):
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         n = self.names
-        return {**self.down.weight_specs(), **(self.out.weight_specs() if self.gate_name else {}),
+        sink = {self.sink_name: WeightSpec((self.heads,), "bias")} if self.sink_name else {}
+        if self.direct:
+            gate = {self.head_gate_name: WeightSpec((self.heads, self.hidden_size))} if self.head_gate_name else {}
+            return {n["q"]: WeightSpec((self.heads * (self.dim + self.rot_dim), self.hidden_size)),
+                    n["dkv"]: WeightSpec((self.row, self.hidden_size)), n["dkv_norm"]: WeightSpec((self.kv_rank,), "norm"),
+                    n["uk"]: WeightSpec((self.heads * self.dim, self.kv_rank)), n["uv"]: WeightSpec((self.heads * self.value_dim, self.kv_rank)),
+                    n["o"]: WeightSpec((self.hidden_size, self.heads * self.value_dim)), **gate, **sink}
+        return {**sink, **self.down.weight_specs(), **(self.out.weight_specs() if self.gate_name else {}),
                 n["dq_norm"]: WeightSpec((self.q_rank,), "norm"), n["dkv_norm"]: WeightSpec((self.kv_rank,), "norm"),
                 n["uq"]: WeightSpec((self.heads * (self.dim + self.rot_dim), self.q_rank)),
                 n["uk"]: WeightSpec((self.heads * self.dim, self.kv_rank)),
@@ -88,8 +117,13 @@ class LatentAttention(Mixer):
     def load(self, weights, rt: Runtime) -> None:
         self.rt = rt
         n, H, d, r, dv, kr = self.names, self.heads, self.dim, self.rot_dim, self.value_dim, self.kv_rank
-        self.down.load(weights, rt)
         self.rotary.load(weights, rt)
+        if self.sink_name:
+            self.sinks = weights.on_device(self.sink_name, torch.float32)
+        if self.direct:
+            self._load_direct(weights, rt)
+            return
+        self.down.load(weights, rt)
         self.q_norm = weights.on_device(n["dq_norm"], torch.float32)
         self.kv_norm = weights.on_device(n["dkv_norm"], torch.float32)
         wide = dict(device=rt.device, dtype=torch.float64)
@@ -111,14 +145,54 @@ class LatentAttention(Mixer):
                 self.up_v_padded[:, :kr] = self.up_v.view(H * dv, kr)
             self.out.load(weights, rt)
             return
-        # the output projection reads the heads' sums of latents: columns W_o,i W_uv,i, zero where a row is padding
-        out = torch.zeros((self.hidden_size, H, self.pad_dim), **wide)
-        out[:, :, :kr] = torch.einsum("ehv,hvk->ehk", o, uv)
-        self.out.load_matrix(out.reshape(self.hidden_size, H * self.pad_dim), rt)
+        self._load_out(o, uv, rt)
+
+    def _load_direct(self, weights, rt: Runtime) -> None:
+        n, H, d, r, dv, kr = self.names, self.heads, self.dim, self.rot_dim, self.value_dim, self.kv_rank
+        wide = dict(device=rt.device, dtype=torch.float64)
+        self.kv_norm = weights.on_device(n["dkv_norm"], torch.float32)
+        q = weights.stored(n["q"]).to(**wide).view(H, d + r, self.hidden_size)
+        dkv = weights.stored(n["dkv"]).to(**wide)
+        uk = weights.stored(n["uk"]).to(**wide).view(H, d, kr)
+        uv = weights.stored(n["uv"]).to(**wide).view(H, dv, kr)
+        order = torch.arange(r, device=rt.device) if self.order is None else self.order.to(rt.device)
+        stack = torch.zeros((self.stack, self.hidden_size), **wide)
+        rows = H * self.row
+        queries = stack[:rows].view(H, self.row, self.hidden_size)
+        queries[:, :kr] = torch.einsum("hdk,hdx->hkx", uk, q[:, :d])
+        queries[:, kr:] = q[:, d:][:, order]
+        stack[rows : rows + kr] = dkv[:kr]
+        stack[rows + kr : rows + self.row] = dkv[kr:][order]
+        if self.head_gate_name:
+            stack[rows + self.row : rows + self.row + H] = weights.stored(self.head_gate_name).to(**wide)
+        self.down.load_matrix(stack, rt)
+        self._load_out(weights.stored(n["o"]).to(**wide).view(self.hidden_size, H, dv), uv, rt)
+
+    def _load_out(self, o, uv, rt: Runtime) -> None:
+        """The output projection on the heads' sums of latents: columns W_o,i W_uv,i, zero where a row is padding."""
+        out = torch.zeros((self.hidden_size, self.heads, self.pad_dim), device=rt.device, dtype=torch.float64)
+        out[:, :, : self.kv_rank] = torch.einsum("ehv,hvk->ehk", o, uv)
+        self.out.load_matrix(out.reshape(self.hidden_size, self.heads * self.pad_dim), rt)
+
+    def _forward_direct(self, x, batch, cache) -> torch.Tensor:
+        ops, rows, amplitude = self.rt.ops, self.heads * self.row, self.rotary.amplitude
+        table = batch.block_tables[cache.group]
+        down = self.down.forward(x, torch.float32)
+        ops.latent_prepare(down[:, rows:], 0, self.kv_rank, self.rot_dim, None, self.kv_norm, self.rotary.inv_freq, self.eps, cache.kv,
+                           table, batch.request_of_token, batch.positions, self.rt.dtype, rot_amplitude=amplitude)
+        q = ops.qkv_rope_write(down, self.heads, 0, self.row, self.row, self.pad_dim, None, None, None, None, self.rotary.inv_freq,
+                               self.kv_rank, self.rot_dim, None, table, batch.request_of_token, batch.positions, self.rt.dtype,
+                               rot_amplitude=amplitude)
+        mixed = ops.paged_attention(q, cache.kv, table, batch, None, self.scale, sinks=self.sinks)
+        if self.head_gate_name:
+            ops.head_gate_(mixed, down[:, rows + self.row : rows + self.row + self.heads], self.heads, self.kv_rank, self.pad_dim)
+        return self.out.forward(mixed, self.out_dtype)
 
     def forward(self, x, batch, cache, write_cache: bool = True) -> torch.Tensor:
         if not write_cache:
             raise ValueError("a latent attention layer fills its own cache")
+        if self.direct:
+            return self._forward_direct(x, batch, cache)
         ops = self.rt.ops
         table = batch.block_tables[cache.group]
         down = self.down.forward(x, torch.float32)
@@ -129,7 +203,7 @@ class LatentAttention(Mixer):
         q = ops.qkv_rope_write(self.up_q.forward(q_latent, torch.float32), self.heads, 0, self.row, self.row, self.pad_dim,
                                None, None, None, None, self.rotary.inv_freq, self.kv_rank, self.rot_dim, None, table,
                                batch.request_of_token, batch.positions, self.rt.dtype, rot_amplitude=amplitude)
-        mixed = ops.paged_attention(q, cache.kv, table, batch, None, self.scale)
+        mixed = ops.paged_attention(q, cache.kv, table, batch, None, self.scale, sinks=self.sinks)
         if self.gate_name:
             gate = down[:, self.q_rank + self.kv_rank + self.rot_dim :]
             mixed = ops.head_linear_gate(mixed.view(mixed.shape[0], -1), self.up_v, self.heads, self.kv_rank, gate,

@@ -84,6 +84,10 @@ def _register_builtin() -> None:
     from .models.fosavik import build_fosavik_plan
 
     register_architecture(FosavikConfig.architecture, FosavikConfig, build_fosavik_plan, replace=True)
+    from .config.damilix import DamilixConfig
+    from .models.damilix import build_damilix_plan
+
+    register_architecture(DamilixConfig.architecture, DamilixConfig, build_damilix_plan, replace=True)
 
 
 _register_builtin()
