@@ -1240,14 +1240,18 @@ def terms_sum(x: torch.Tensor, routed: Optional[torch.Tensor], sorted_rows: Opti
 
 
 def linear_grouped(x: torch.Tensor, weight, groups: int, tile_group: torch.Tensor, out_dtype: torch.dtype = torch.bfloat16,
-                   relu2: bool = False, gated: Optional[tuple] = None) -> torch.Tensor:
+                   relu2: bool = False, gated: Optional[tuple] = None, rows_a_group: Optional[int] = None) -> torch.Tensor:
     """Rows sorted by group times one of ``groups`` stacked matrices each: ``x`` [tiles * 128, K] (bfloat16), ``weight``
     [groups * N, K] (row-major, or a ``TiledWeight`` with N a multiple of 128), ``tile_group`` [tiles] the matrix of each
     128-row tile.  Returns [tiles * 128, N]; with ``relu2`` relu(product)^2 (bfloat16).  ``gated`` = (activation, limit,
     slope): every matrix holds 8 gate rows, their 8 up rows, 8 gate rows, ... and the result is act(gate) * up,
-    [tiles * 128, N / 2] (bfloat16), the activations those of ``gated_activation``."""
+    [tiles * 128, N / 2] (bfloat16), the activations those of ``gated_activation``.  ``rows_a_group`` N: further rows
+    may stand behind the groups' in ``weight``, which are left alone (None: all rows are the groups')."""
     m, k, total = _check_product(x, weight)
     _need_cuda(tile_group)
+    if rows_a_group is not None:
+        assert total >= groups * rows_a_group
+        total = groups * rows_a_group
     assert total % groups == 0 and m % 128 == 0 and tile_group.dtype == torch.int32 and tile_group.numel() == m // 128
     n = total // groups
     tiled = isinstance(weight, TiledWeight)

@@ -204,9 +204,10 @@ class RoutedExperts(FeedForward):
         tile_group, slot_of, row_of_slot = ops.route_plan(ids, self.experts)
         rows = ops.route_gather(x, row_of_slot)
         if self.gated and self.interleaved:
-            hidden = ops.linear_grouped(rows, self.up.weight, self.experts, tile_group, gated=(self.gate_act, self.limit, self.slope))
+            hidden = ops.linear_grouped(rows, self.up.weight, self.experts, tile_group, gated=(self.gate_act, self.limit, self.slope),
+                                        rows_a_group=2 * self.expert_size)
         elif self.gated:
-            hidden = ops.gated_activation(ops.linear_grouped(rows, self.up.weight, self.experts, tile_group), self.gate_act,
+            hidden = ops.gated_activation(ops.linear_grouped(rows, self.up.weight, self.experts, tile_group, rows_a_group=2 * self.expert_size), self.gate_act,
                                           self.limit, self.slope)
         else:
             hidden = ops.linear_grouped(rows, self.up.weight, self.experts, tile_group, relu2=True)
