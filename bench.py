@@ -358,6 +358,30 @@ def fosavik_config(size: dict, layers: int, intermediate: int) -> dict:
             "norm": {"eps": 1e-6}, "layers": out}
 
 
+DAMILIX_IDENTITY = 2     # experts of the router that hand their input on
+DAMILIX_SIDE = 256       # columns of a token's own input per layer
+
+
+def damilix_config(size: dict, layers: int, intermediate: int) -> dict:
+    """A Damilix config.json of one size: layers in the order latent attention (neighbouring columns rotated, frequencies
+    stretched by index), gated linear attention, latent attention (halves rotated), gated linear attention (and so on); latent
+    attention with 16 heads over a cached row of 256 columns, as in the Bikilix configuration; the linear attention with the
+    heads of the Figalix configuration's matrix memory; the first layer of four with a dense gated feed-forward as large as the
+    dense model's, the others with the size's experts, two identity experts and a shared branch as large as one expert; an input
+    of the token's own of 256 columns a layer."""
+    width = size["width"]
+    lat = dict(BIKILIX_LATENT, scale=(BIKILIX_LATENT["dim"] + BIKILIX_LATENT["rot_dim"]) ** -0.5,
+               rot={"base": 500000.0, "dims": BIKILIX_LATENT["rot_dim"]})
+    stretched = dict(lat, rot=dict(lat["rot"], scaling={"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}))
+    linear = {"heads": width // 256, "dim": FIGALIX_MEMORY["dim"], "vdim": FIGALIX_MEMORY["vdim"], "tau": 16.0}
+    mixers = [("latent_attention", stretched), ("gla", linear), ("latent_attention_2", lat), ("gla", linear)]
+    experts = {"kind": "moe", "expert": {"ff": size["ff"]}, "shared": {"ff": size["ff"]},
+               "router": {"experts": size["experts"], "identity": DAMILIX_IDENTITY, "top": size["top"], "scale": 1.0}}
+    mlps = [{"kind": "dense", "ff": intermediate}, experts, experts, experts]
+    return {"architecture": "Damilix", "width": width, "vocab": size["vocab"], "norm": {"eps": 1e-6}, "token_side": {"dim": DAMILIX_SIDE},
+            "layers": [{"type": mixers[i % 4][0], "mixer": dict(mixers[i % 4][1]), "mlp": dict(mlps[i % 4])} for i in range(layers)]}
+
+
 def design_configs(size: dict, layers: int):
     """(Zoferax config.json, Qwen3 config.json, Silupel config.json and so on) of one size: the same width, heads and layer count;
     the dense feed-forward is as large as the experts that one token uses (3 I H = 2 top ff H)."""
@@ -372,7 +396,7 @@ def design_configs(size: dict, layers: int):
                  rope_theta=1000000.0, tie_word_embeddings=False)
     return {"zoferax": zoferax, "qwen3-dense": dense, "silupel": silupel_config(size, layers, intermediate),
             "figalix": figalix_config(size, layers, intermediate), "bikilix": bikilix_config(size, layers, intermediate),
-            "fosavik": fosavik_config(size, layers, intermediate)}
+            "fosavik": fosavik_config(size, layers, intermediate), "damilix": damilix_config(size, layers, intermediate)}
 
 
 def _kernel_rows(summary: dict, tokens: int, context_pairs: float, cache_rows: float, size: dict, design: str, peaks,
@@ -383,7 +407,7 @@ def _kernel_rows(summary: dict, tokens: int, context_pairs: float, cache_rows: f
     import re
 
     width, heads, kvh, dk = size["width"], size["heads"], size["kv_heads"], size["dim"]
-    dv = size["vdim"] if design in ("zoferax", "silupel", "figalix", "bikilix") else dk  # (fosavik: values of the size's key width)
+    dv = size["vdim"] if design in ("zoferax", "silupel", "figalix", "bikilix", "damilix") else dk  # (fosavik: values of the size's key width)
     visible = visible or (lambda mask: (context_pairs, cache_rows))
     routed = size["experts"] * size["ff"]
     rows = []
@@ -413,6 +437,13 @@ def _kernel_rows(summary: dict, tokens: int, context_pairs: float, cache_rows: f
         elif match:
             m, n, k, form = map(int, match.groups())
             flops, bytes_ = 2.0 * m * n * k, 2.0 * (m * k + n * k) + m * (n // 2 if form == 2 else n) * (4 if form in (1, 3) else 2)
+            if design == "damilix" and (n == 2 * (routed + size["ff"]) or k == routed + size["ff"]):
+                # the experts and the branch that every token runs, stacked: a token needs top of the ones and the other whole
+                share = (size["top"] * size["experts"] / (size["experts"] + DAMILIX_IDENTITY) + 1) / (size["experts"] + 1)
+                flops *= share
+                hidden_in = share if k == routed + size["ff"] else 1
+                bytes_ = 2.0 * m * k * hidden_in + 2.0 * n * k * min(1.0, share * max(1, m)) + m * n * (4.0 if form == 1 else 2.0 * share)
+                label += " (experts and the shared branch; work = the chosen experts' and its own)"
             if design in ("zoferax", "bikilix") and (routed in (n, k) or 2 * routed == n):  # the experts: a token needs top of them
                 share = size["top"] / size["experts"]
                 flops *= share
@@ -423,7 +454,7 @@ def _kernel_rows(summary: dict, tokens: int, context_pairs: float, cache_rows: f
             # a launch that says its shape: pairs and cache rows of the keys that its mask lets a query see
             a_heads, a_kv, a_d, a_mask = (int(v) for v in re.search(r"heads=(\d+) kv=(\d+) d=(\d+) mask=(-?\d+)", name).groups())
             pairs, rows_read = visible(a_mask)
-            shared = 1.0 if (design in ("silupel", "bikilix") and a_kv == 1) else 2.0  # a latent row is key and value in one
+            shared = 1.0 if (design in ("silupel", "bikilix", "damilix") and a_kv == 1) else 2.0  # a latent row is key and value in one
             flops = 2.0 * a_heads * 2 * a_d * pairs * count
             if design == "fosavik" and a_mask == 0:  # a map's own half of the key row, and the whole value row
                 flops *= 0.75
@@ -431,6 +462,25 @@ def _kernel_rows(summary: dict, tokens: int, context_pairs: float, cache_rows: f
         elif "attention" in name:
             flops = 2.0 * heads * (dk + dv) * context_pairs * count
             bytes_ = (2.0 * kvh * (dk + dv) * cache_rows + 2.0 * tokens * heads * (dk + dv)) * count
+        elif "channel_walk" in name:
+            # as the matrix memory's walk, with a decay per key column
+            cells = (width // 256) * FIGALIX_MEMORY["dim"] * FIGALIX_MEMORY["vdim"]
+            cols = (width // 256) * (2 * FIGALIX_MEMORY["dim"] + 2 * FIGALIX_MEMORY["vdim"]) + 16
+            simt = 6.0 * tokens * cells * count
+            bytes_ = (4.0 * tokens * cols + 2.0 * tokens * width + 8.0 * cells * requests) * count
+        elif "channel_chunks" in name:
+            # as the matrix memory's chunks
+            s_heads, s_d, s_dv = width // 256, FIGALIX_MEMORY["dim"], FIGALIX_MEMORY["vdim"]
+            simt = tokens * s_heads * (64.0 * (s_d + s_dv) + 4.0 * s_d * s_dv) * count
+            bytes_ = (4.0 * tokens * s_heads * (2 * s_d + 2 * s_dv) + 8.0 * s_heads * s_d * s_dv * requests) * count
+        elif "terms_norm_add" in name:
+            # the stream in and out, its copy, the routed rows (few tokens: summed, 32-bit; else the chosen ones in bfloat16)
+            few = tokens * size["top"] < 512
+            bytes_ = tokens * width * (10.0 + (4.0 if few else 2.0 * size["top"] + 4.0)) * count
+        elif "token_gate" in name:
+            bytes_ = tokens * DAMILIX_SIDE * 8.0 * count
+        elif "embedding_norm" in name:
+            bytes_ = tokens * width * 8.0 * count
         elif "head_major" in name or "head_gate_rows" in name:
             bytes_ = tokens * BIKILIX_LATENT["heads"] * (4.0 * (BIKILIX_LATENT["kv_rank"] + BIKILIX_LATENT["rot_dim"]) if "major" in name
                                                           else 10.0 * BIKILIX_LATENT["vdim"]) * count
@@ -489,15 +539,17 @@ def _kernel_rows(summary: dict, tokens: int, context_pairs: float, cache_rows: f
         elif "real_gated_scan" in name:
             bytes_ = (tokens * width * 18.0 + requests * width * 8.0) * count
         elif "gated_group_norm" in name:
-            bytes_ = tokens * 2 * width * 10.0 * count
+            bytes_ = tokens * (1 if design == "damilix" else 2) * width * 10.0 * count
         elif "rms_pair_mean" in name:
             bytes_ = tokens * width * 12.0 * count
         elif "add_dyt" in name or "add_scaled" in name:
             bytes_ = tokens * width * 16.0 * count
+        elif "head_gate" in name and design == "damilix":
+            bytes_ = tokens * BIKILIX_LATENT["heads"] * BIKILIX_LATENT["kv_rank"] * 4.0 * count
         elif "head_gate" in name:
             bytes_ = tokens * heads * dv * 4.0 * count
         elif "gated_expert_gate" in name:
-            bytes_ = tokens * routed * 6.0 * count
+            bytes_ = tokens * (routed + (size["ff"] if design == "damilix" else 0)) * 6.0 * count
         elif "qkv_wide_norm" in name:
             cols = heads * dk + kvh * (dk + dv)
             bytes_ = tokens * (4.0 * cols + 2.0 * cols) * count
@@ -676,7 +728,7 @@ def main() -> int:
                              "equal layer sizes (--sizes), with every step's time by kernel; a line of its own.")
     parser.add_argument("--sizes", default="2k,4k", help="layer sizes of --workload designs: " + ", ".join(DESIGN_SIZES))
     parser.add_argument("--designs", default="zoferax,qwen3-dense",
-                        help="which designs --workload designs measures, comma separated: zoferax, silupel, figalix, bikilix, fosavik, qwen3-dense")
+                        help="which designs --workload designs measures, comma separated: zoferax, silupel, figalix, bikilix, fosavik, damilix, qwen3-dense")
     args = parser.parse_args()
 
     if args.impl == "reference":
