@@ -145,6 +145,60 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, long y_stri
     }
 }
 
+// A warp per (row, group) with 16-byte loads, the row in registers (group width a multiple of 4 below 512; aligned rows).
+template <typename O>
+__global__ void __launch_bounds__(256) gated_group_norm_warp_kernel(const float* __restrict__ y, long y_stride, const float* __restrict__ gate,
+                                                                    long g_stride, const float* __restrict__ weight, float eps,
+                                                                    O* __restrict__ out, long rows, int groups, int group_width, int mode) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const long unit = blockIdx.x * (long)(blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (unit >= rows * groups) return;
+    const long row = unit / groups;
+    const int c0 = (int)(unit - row * groups) * group_width;
+    const float* py = y + row * y_stride + c0;
+    const float* pg = gate + row * g_stride + c0;
+    float4 v[4], g[4];
+    float sum = 0.0f;
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+        const int c = (lane + n * 32) * 4;
+        if (c >= group_width) break;
+        v[n] = *reinterpret_cast<const float4*>(py + c);
+        g[n] = *reinterpret_cast<const float4*>(pg + c);
+    }
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+        if ((lane + n * 32) * 4 >= group_width) break;
+        float4 f;
+        if (mode == 1) f = make_float4(sf_sigmoid(g[n].x), sf_sigmoid(g[n].y), sf_sigmoid(g[n].z), sf_sigmoid(g[n].w));
+        else f = make_float4(sf_silu(g[n].x), sf_silu(g[n].y), sf_silu(g[n].z), sf_silu(g[n].w));
+        const float4 gated = make_float4(v[n].x * f.x, v[n].y * f.y, v[n].z * f.z, v[n].w * f.w);
+        const float4 counted = mode == 0 ? gated : v[n];
+        sum += (counted.x * counted.x + counted.y * counted.y) + (counted.z * counted.z + counted.w * counted.w);
+        v[n] = gated;
+    }
+    const float r = rsqrtf(warp_sum(sum) / (float)group_width + eps);
+    O* po = out + row * (long)groups * group_width + c0;
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+        const int c = (lane + n * 32) * 4;
+        if (c >= group_width) break;
+        const float4 w = *reinterpret_cast<const float4*>(weight + c0 + c);
+        const float a = v[n].x * r * w.x, b = v[n].y * r * w.y, d = v[n].z * r * w.z, e = v[n].w * r * w.w;
+        if (sizeof(O) == 4) {
+            *reinterpret_cast<float4*>(po + c) = make_float4(a, b, d, e);
+        } else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(d, e);
+            uint2 packed;
+            packed.x = *reinterpret_cast<const uint32_t*>(&lo);
+            packed.y = *reinterpret_cast<const uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>(po + c) = packed;
+        }
+    }
+}
+
 // The same with 16-byte loads, a block of up to 1,024 threads per (row, group), the gated values in registers between the
 // statistics and the output (group width a multiple of 4, at most 4 * VEC * blockDim values; aligned rows).
 template <typename O, int VEC>
@@ -203,8 +257,12 @@ static int gated_group_norm_launch(const float* y, long y_stride, const float* g
     if (rows <= 0) return 0;
     if (groups <= 0 || group_width <= 0 || mode < 0 || mode > 2) return KIRAI_ERR_BAD_SIZE;
     const long units = (long)rows * groups;
-    const bool vec = group_width % 4 == 0 && group_width >= 512 && group_width <= 4 * 4 * 1024 && y_stride % 4 == 0 && g_stride % 4 == 0 &&
-                     (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+    const bool aligned = group_width % 4 == 0 && y_stride % 4 == 0 && g_stride % 4 == 0 &&
+                         (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+    const bool vec = aligned && group_width >= 512 && group_width <= 4 * 4 * 1024;
+    if (aligned && group_width < 512)
+        return launch_pdl(gated_group_norm_warp_kernel<O>, dim3((unsigned)((units + 7) / 8)), dim3(256), 0, stream, 1u, y, y_stride, gate,
+                          g_stride, weight, eps, (O*)out, (long)rows, groups, group_width, mode);
     if (vec) {
         // many units: four pieces a thread; few: one or two, so that a row's loads are all in flight at once
         const int quads = group_width / 4;

@@ -76,22 +76,25 @@ KIRAI_EXPORT int kirai_embedding_norm_bf16(const void* table, const int* ids, co
 }
 
 // out [T, dim] = gelu_tanh(z [T, dim]) * table[id, first .. first + dim); table rows have `row` numbers.
-template <typename T>
+template <typename T, int VEC>
 __global__ void token_gate_kernel(const float* __restrict__ z, const T* __restrict__ table, const int* __restrict__ ids, T* __restrict__ out,
                                   long tokens, int dim, long row, long first, int vocab, int* __restrict__ error_flag) {
     pdl_launch_dependents();
     pdl_wait();
-    const long total = tokens * dim;
-    for (long at = blockIdx.x * (long)blockDim.x + threadIdx.x; at < total; at += (long)gridDim.x * blockDim.x) {
+    const long total = tokens * dim / VEC;
+    for (long item = blockIdx.x * (long)blockDim.x + threadIdx.x; item < total; item += (long)gridDim.x * blockDim.x) {
+        const long at = item * VEC;
         const long token = at / dim;
         const int c = (int)(at - token * dim);
         const int id = ids[token];
-        if (id < 0 || id >= vocab) {
-            atomicExch(error_flag, KIRAI_FLAG_BAD_TOKEN);
-            out[at] = from_f32<T>(0.0f);
-            continue;
-        }
-        out[at] = from_f32<T>(sf_gelu_tanh(z[at]) * to_f32<T>(table[(size_t)id * row + first + c]));
+        const bool known = id >= 0 && id < vocab;
+        if (!known) atomicExch(error_flag, KIRAI_FLAG_BAD_TOKEN);
+        const T* e = table + (size_t)(known ? id : 0) * row + first + c;
+        T values[VEC];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) values[j] = from_f32<T>(known ? sf_gelu_tanh(z[at + j]) * to_f32<T>(e[j]) : 0.0f);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) out[at + j] = values[j];
     }
 }
 
@@ -100,9 +103,14 @@ static int token_gate_launch(const float* z, const void* table, const int* ids, 
                              int* error_flag, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (dim <= 0 || first < 0 || first + dim > row || vocab <= 0) return KIRAI_ERR_BAD_SIZE;
-    const long total = (long)tokens * dim;
+    // two columns a thread where a row has enough of them, so that a block has several rows' loads in flight
+    const bool pairs = dim % 2 == 0 && tokens >= 64;
+    const long total = (long)tokens * dim / (pairs ? 2 : 1);
     const unsigned blocks = (unsigned)min((total + 255) / 256, (long)148 * 16);
-    return launch_pdl(token_gate_kernel<T>, dim3(blocks), dim3(256), 0, stream, 1u, z, (const T*)table, ids, (T*)out, (long)tokens, dim, row, first,
+    if (pairs)
+        return launch_pdl(token_gate_kernel<T, 2>, dim3(blocks), dim3(256), 0, stream, 1u, z, (const T*)table, ids, (T*)out, (long)tokens, dim, row,
+                          first, vocab, error_flag);
+    return launch_pdl(token_gate_kernel<T, 1>, dim3(blocks), dim3(256), 0, stream, 1u, z, (const T*)table, ids, (T*)out, (long)tokens, dim, row, first,
                       vocab, error_flag);
 }
 
