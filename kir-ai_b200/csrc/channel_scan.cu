@@ -200,17 +200,26 @@ __global__ void __launch_bounds__(THREADS) channel_prepare_kernel(const ChannelS
 }
 
 // ------------------------------------------------------------------------------------------------ the chunks' products
-// The tiles of a block: q [d][64], k [d][64], P [64][64] as channel_prepare left them, v [64][cp], the state [d][cp], e^(G_last).
+// The tiles of a block, in this order as far as its kernel has them: q [d][64], k [d][64], P [64][64] as channel_prepare left
+// them, v [64][cp], the state [d][cp], e^(G_last) [d].  A thread's columns are J tx .. J tx + J - 1 of cp = 16 J.
+enum Kind { CHAIN, SHARE, READ };
+
 struct Tiles {
     float *Q, *K, *P, *V, *S, *kept;
-    __device__ Tiles(float* smem, int d, int cp) {
-        Q = smem, K = Q + (long)d * CHUNK, P = K + (long)d * CHUNK, V = P + CHUNK * CHUNK, S = V + CHUNK * cp, kept = S + (long)d * cp;
+    __device__ Tiles(float* smem, int d, int cp, Kind kind) {
+        Q = smem;
+        K = Q + (kind == SHARE ? 0L : (long)d * CHUNK);
+        P = K + (kind == READ ? 0L : (long)d * CHUNK);
+        V = P + (kind == SHARE ? 0 : CHUNK * CHUNK);
+        S = V + CHUNK * cp;
+        kept = S + (long)d * cp;
     }
 };
 
-__host__ __device__ inline long product_floats(int d, int cols) {
+__host__ __device__ inline long product_floats(int d, int cols, Kind kind) {
     const int cp = cols_pitch(cols);
-    return 2L * d * CHUNK + (long)CHUNK * CHUNK + (long)CHUNK * cp + (long)d * cp + d;
+    const long tile = (long)d * CHUNK, square = (long)CHUNK * CHUNK, v = (long)CHUNK * cp, state = (long)d * cp;
+    return kind == CHAIN ? 2 * tile + square + v + state + d : kind == SHARE ? tile + v : tile + square + v + state;
 }
 
 __device__ __forceinline__ void copy_async16(float* to, const float* from) {
@@ -220,7 +229,53 @@ __device__ __forceinline__ void fetch_flat(float* to, const float* from, long fl
     for (long i = threadIdx.x * 4L; i < floats; i += THREADS * 4L) copy_async16(to + i, from + i);
 }
 
-// o of tokens t = 4 ty + i at columns tx + 16 j.
+// `live` of `rows` rows of `cols` columns (row stride `stride`) into a tile [rows][cp], zero elsewhere; 16 bytes a copy where
+// the rows allow it.
+__device__ __forceinline__ void fetch_rows(float* to, int cp, const float* from, long stride, int live, int rows, int cols) {
+    if (cols == cp && stride % 4 == 0 && ((uintptr_t)from & 15) == 0) {
+        const int quads = cp / 4;
+        for (int i = threadIdx.x; i < rows * quads; i += THREADS) {
+            const int r = i / quads, c = 4 * (i - r * quads);
+            if (r < live) copy_async16(to + r * cp + c, from + r * stride + c);
+            else *reinterpret_cast<float4*>(to + r * cp + c) = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < rows * cp; i += THREADS) {
+        const int r = i / cp, c = i - r * cp;
+        if (r < live && c < cols) copy_async(to + i, from + r * stride + c);
+        else to[i] = 0.0f;
+    }
+}
+
+// A thread's J neighbouring columns of a tile's row.
+template <int J>
+__device__ __forceinline__ void columns(const float* row, int tx, float (&x)[J]) {
+    if (J == 4) {
+        const float4 v = *reinterpret_cast<const float4*>(row + 4 * tx);
+        x[0] = v.x, x[1 % J] = v.y, x[2 % J] = v.z, x[3 % J] = v.w;
+    } else if (J == 2) {
+        const float2 v = *reinterpret_cast<const float2*>(row + 2 * tx);
+        x[0] = v.x, x[1 % J] = v.y;
+    } else {
+#pragma unroll
+        for (int j = 0; j < J; ++j) x[j] = row[J * tx + j];
+    }
+}
+
+// The same columns to global memory, those below `cols` only.
+template <int J>
+__device__ __forceinline__ void store_columns(float* row, int tx, int cols, const float (&x)[J]) {
+    if (J == 4 && 4 * tx + 4 <= cols && ((uintptr_t)(row + 4 * tx) & 15) == 0) {
+        *reinterpret_cast<float4*>(row + 4 * tx) = make_float4(x[0], x[1 % J], x[2 % J], x[3 % J]);
+        return;
+    }
+#pragma unroll
+    for (int j = 0; j < J; ++j)
+        if (J * tx + j < cols) row[J * tx + j] = x[j];
+}
+
+// o of tokens t = 4 ty + i at the thread's columns.
 template <int J>
 __device__ __forceinline__ void read_out(const ChannelScan& a, const Tiles& w, int head, int col0, int cols, long row0, int len) {
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4, d = a.d;
@@ -230,71 +285,73 @@ __device__ __forceinline__ void read_out(const ChannelScan& a, const Tiles& w, i
     for (int c = 0; c < d; ++c) {
         const float4 qv = *reinterpret_cast<const float4*>(w.Q + c * CHUNK + 4 * ty);
         const float qs[4] = {qv.x, qv.y, qv.z, qv.w};
+        float sv[J];
+        columns<J>(w.S + c * cp, tx, sv);
 #pragma unroll
-        for (int j = 0; j < J; ++j) {
-            const float sv = w.S[c * cp + tx + 16 * j];
+        for (int j = 0; j < J; ++j)
 #pragma unroll
-            for (int i = 0; i < 4; ++i) o[i][j] = fmaf(qs[i], sv, o[i][j]);
-        }
+            for (int i = 0; i < 4; ++i) o[i][j] = fmaf(qs[i], sv[j], o[i][j]);
     }
     const int s_end = min(4 * ty + 4, len);
 #pragma unroll 4
     for (int s = 0; s < s_end; ++s) {
         const float4 pv = *reinterpret_cast<const float4*>(w.P + s * CHUNK + 4 * ty);
         const float ps[4] = {pv.x, pv.y, pv.z, pv.w};
+        float vv[J];
+        columns<J>(w.V + s * cp, tx, vv);
 #pragma unroll
-        for (int j = 0; j < J; ++j) {
-            const float vv = w.V[s * cp + tx + 16 * j];
+        for (int j = 0; j < J; ++j)
 #pragma unroll
-            for (int i = 0; i < 4; ++i) o[i][j] = fmaf(ps[i], vv, o[i][j]);
-        }
+            for (int i = 0; i < 4; ++i) o[i][j] = fmaf(ps[i], vv[j], o[i][j]);
     }
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const int t = 4 * ty + i;
-        if (t >= len) continue;
-#pragma unroll
-        for (int j = 0; j < J; ++j)
-            if (tx + 16 * j < cols) a.out[(row0 + t) * ((long)a.heads * a.dv) + (long)head * a.dv + col0 + tx + 16 * j] = o[i][j];
+        if (t < len) store_columns<J>(a.out + (row0 + t) * ((long)a.heads * a.dv) + (long)head * a.dv + col0, tx, cols, o[i]);
     }
 }
 
-// S <- diag(kept) S + k v^T over the chunk's tokens; `fresh`: the state before it is zero.
-template <int J>
-__device__ __forceinline__ void update(const Tiles& w, int d, int len, bool fresh) {
+// sum_s k_s v_s^T over the chunk's tokens, R state rows a thread at a time, handed row by row to `take(row, sums)`.
+template <int J, int R, typename Take>
+__device__ __forceinline__ void outer_products(const Tiles& w, int d, int len, Take take) {
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     constexpr int cp = 16 * J;
-    for (int r0 = 0; r0 < d; r0 += 64) {
-        float acc[4][J] = {};
-        const int c0 = r0 + 4 * ty;
+    for (int r0 = 0; r0 < d; r0 += 16 * R) {
+        float acc[R][J] = {};
+        const int c0 = r0 + R * ty;
         const int quads = (len + 3) / 4;  // (tokens behind the last hold zeros)
         for (int s4 = 0; s4 < quads; ++s4) {
-            float4 kv[4];
+            float4 kv[R];
 #pragma unroll
-            for (int i = 0; i < 4; ++i)
+            for (int i = 0; i < R; ++i)
                 kv[i] = c0 + i < d ? *reinterpret_cast<const float4*>(w.K + (c0 + i) * CHUNK + 4 * s4) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                float ks[4];
+                float vv[J];
+                columns<J>(w.V + (4 * s4 + e) * cp, tx, vv);
 #pragma unroll
-                for (int i = 0; i < 4; ++i) ks[i] = e == 0 ? kv[i].x : e == 1 ? kv[i].y : e == 2 ? kv[i].z : kv[i].w;
+                for (int i = 0; i < R; ++i) {
+                    const float k = e == 0 ? kv[i].x : e == 1 ? kv[i].y : e == 2 ? kv[i].z : kv[i].w;
 #pragma unroll
-                for (int j = 0; j < J; ++j) {
-                    const float vv = w.V[(4 * s4 + e) * cp + tx + 16 * j];
-#pragma unroll
-                    for (int i = 0; i < 4; ++i) acc[i][j] = fmaf(ks[i], vv, acc[i][j]);
+                    for (int j = 0; j < J; ++j) acc[i][j] = fmaf(k, vv[j], acc[i][j]);
                 }
             }
         }
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
-#pragma unroll
-            for (int j = 0; j < J; ++j)
-                if (c0 + i < d) {
-                    float* at = w.S + (c0 + i) * cp + tx + 16 * j;
-                    *at = fresh ? acc[i][j] : fmaf(w.kept[c0 + i], *at, acc[i][j]);
-                }
+        for (int i = 0; i < R; ++i)
+            if (c0 + i < d) take(c0 + i, acc[i]);
     }
+}
+
+// S <- diag(kept) S + sum_s k_s v_s^T in shared memory.
+template <int J>
+__device__ __forceinline__ void update(const Tiles& w, int d, int len) {
+    const int tx = threadIdx.x & 15;
+    outer_products<J, 4>(w, d, len, [&](int c, const float(&sums)[J]) {
+        float* at = w.S + c * 16 * J + J * tx;
+#pragma unroll
+        for (int j = 0; j < J; ++j) at[j] = fmaf(w.kept[c], at[j], sums[j]);
+    });
 }
 
 template <int J>
@@ -304,7 +361,7 @@ __global__ void __launch_bounds__(THREADS) channel_chain_kernel(const ChannelSca
     const int request = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * a.cols, d = a.d, tid = threadIdx.x;
     const int cols = min(a.cols, a.dv - col0);
     constexpr int cp = 16 * J;
-    const Tiles w(smem, d, cp);
+    const Tiles w(smem, d, cp, CHAIN);
     const long first = a.query_start[request];
     const int count = (int)(a.query_start[request + 1] - first);
     const int slot = a.slots[request];
@@ -320,7 +377,7 @@ __global__ void __launch_bounds__(THREADS) channel_chain_kernel(const ChannelSca
     const float* v_from = a.v + (long)head * a.dv + col0;
     auto tile_of = [&](int chunk) { return a.tiles + ((long)(before + chunk) * a.heads + head) * tile_floats; };
     fetch_flat(w.Q, tile_of(0), tile_floats);
-    fetch_along(w.V, v_from + first * a.stride, a.stride, min(CHUNK, count), cols, cp);
+    fetch_rows(w.V, cp, v_from + first * a.stride, a.stride, min(CHUNK, count), CHUNK, cols);
     for (int c0 = 0; c0 < count; c0 += CHUNK) {
         const int len = min(CHUNK, count - c0), chunk = c0 / CHUNK;
         const int next_len = min(CHUNK, count - c0 - CHUNK);  // <= 0: this chunk is the last
@@ -333,11 +390,11 @@ __global__ void __launch_bounds__(THREADS) channel_chain_kernel(const ChannelSca
             fetch_flat(w.Q, tile_of(chunk + 1), (long)d * CHUNK);
             fetch_flat(w.P, tile_of(chunk + 1) + 2L * d * CHUNK, CHUNK * CHUNK);
         }
-        update<J>(w, d, len, false);
+        update<J>(w, d, len);
         __syncthreads();
         if (next_len > 0) {
             fetch_flat(w.K, tile_of(chunk + 1) + (long)d * CHUNK, (long)d * CHUNK);
-            fetch_along(w.V, v_from + (first + c0 + CHUNK) * a.stride, a.stride, next_len, cols, cp);
+            fetch_rows(w.V, cp, v_from + (first + c0 + CHUNK) * a.stride, a.stride, next_len, CHUNK, cols);
         }
     }
     for (int i = tid; i < d * cp; i += THREADS) {
@@ -350,26 +407,23 @@ template <int J>
 __global__ void __launch_bounds__(THREADS) channel_share_kernel(const ChannelScan a) {
     extern __shared__ __align__(16) float smem[];
     pdl_launch_dependents();
-    const int head = blockIdx.y, col0 = blockIdx.z * a.cols, d = a.d;
+    const int head = blockIdx.y, col0 = blockIdx.z * a.cols, d = a.d, tx = threadIdx.x & 15;
     const int cols = min(a.cols, a.dv - col0);
     constexpr int cp = 16 * J;
-    const Tiles w(smem, d, cp);
+    const Tiles w(smem, d, cp, SHARE);
     ChunkPlace at;
     const bool found = find_chunk(a.query_start, a.requests, blockIdx.x, at);
     pdl_wait();
     if (!found) return;
     const long unit = (long)blockIdx.x * a.heads + head;
     fetch_flat(w.K, a.tiles + unit * (2L * d + CHUNK) * CHUNK + (long)d * CHUNK, (long)d * CHUNK);
-    fetch_along(w.V, a.v + (long)head * a.dv + col0 + at.row0 * a.stride, a.stride, at.len, cols, cp);
+    fetch_rows(w.V, cp, a.v + (long)head * a.dv + col0 + at.row0 * a.stride, a.stride, at.len, CHUNK, cols);
     copies_wait();
     __syncthreads();
-    update<J>(w, d, at.len, true);
-    __syncthreads();
     float* U = a.share + unit * d * a.dv + col0;
-    for (int i = threadIdx.x; i < d * cp; i += THREADS) {
-        const int c = i / cp, j = i - c * cp;
-        if (j < cols) U[(long)c * a.dv + j] = w.S[i];
-    }
+    const auto keep = [&](int c, const float(&sums)[J]) { store_columns<J>(U + (long)c * a.dv, tx, cols, sums); };
+    if (d > 64) outer_products<J, 8>(w, d, at.len, keep);
+    else outer_products<J, 4>(w, d, at.len, keep);
 }
 
 // Block (request, head, run of 256 entries of the state): the state at every chunk's start takes the place of the chunk's own share.
@@ -403,7 +457,7 @@ __global__ void __launch_bounds__(THREADS) channel_out_kernel(const ChannelScan 
     const int head = blockIdx.y, col0 = blockIdx.z * a.cols, d = a.d;
     const int cols = min(a.cols, a.dv - col0);
     constexpr int cp = 16 * J;
-    const Tiles w(smem, d, cp);
+    const Tiles w(smem, d, cp, READ);
     ChunkPlace at;
     const bool found = find_chunk(a.query_start, a.requests, blockIdx.x, at);
     const int slot = found ? a.slots[at.request] : -1;
@@ -413,13 +467,8 @@ __global__ void __launch_bounds__(THREADS) channel_out_kernel(const ChannelScan 
     const float* tile = a.tiles + unit * (2L * d + CHUNK) * CHUNK;
     fetch_flat(w.Q, tile, (long)d * CHUNK);
     fetch_flat(w.P, tile + 2L * d * CHUNK, CHUNK * CHUNK);
-    fetch_along(w.V, a.v + (long)head * a.dv + col0 + at.row0 * a.stride, a.stride, at.len, cols, cp);
-    const float* U = a.share + unit * d * a.dv + col0;
-    for (int i = threadIdx.x; i < d * cp; i += THREADS) {
-        const int c = i / cp, j = i - c * cp;
-        if (j < cols) copy_async(w.S + i, U + (long)c * a.dv + j);
-        else w.S[i] = 0.0f;
-    }
+    fetch_rows(w.V, cp, a.v + (long)head * a.dv + col0 + at.row0 * a.stride, a.stride, at.len, CHUNK, cols);
+    fetch_rows(w.S, cp, a.share + unit * d * a.dv + col0, a.dv, d, d, cols);
     copies_wait();
     __syncthreads();
     read_out<J>(a, w, head, col0, cols, at.row0, at.len);
@@ -427,24 +476,21 @@ __global__ void __launch_bounds__(THREADS) channel_out_kernel(const ChannelScan 
 
 // How many value columns a block takes: as many as fit shared memory, fewer (16 at least) while the grid would leave most of
 // the device idle.  0 when even 16 do not fit.
-int choose_cols(long groups, int d, int dv, bool side_by_side, long* bytes) {
-    int device = 0, limit = 0, sms = 0, all = 0;
+int choose_cols(long groups, int d, int dv, bool side_by_side) {
+    int device = 0, limit = 0, sms = 0;
     if (cudaGetDevice(&device) != cudaSuccess ||
         cudaDeviceGetAttribute(&limit, cudaDevAttrMaxSharedMemoryPerBlockOptin, device) != cudaSuccess ||
-        cudaDeviceGetAttribute(&all, cudaDevAttrMaxSharedMemoryPerMultiprocessor, device) != cudaSuccess ||
         cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device) != cudaSuccess)
         return 0;
+    const Kind kind = side_by_side ? READ : CHAIN;
     int cols = dv < 64 ? dv : 64;
-    while (side_by_side && cols > 32 && 2 * (product_floats(d, cols) * 4 + 1024) > all) cols -= 16;
-    while (cols > 16 && (product_floats(d, cols) * 4 > limit || groups * ((dv + cols - 1) / cols) < sms)) cols = cols > 32 ? cols - 16 : 16;
-    *bytes = product_floats(d, cols) * 4;
-    return *bytes <= limit ? cols : 0;
+    while (cols > 16 && (product_floats(d, cols, kind) * 4 > limit || groups * ((dv + cols - 1) / cols) < sms)) cols = cols > 32 ? cols - 16 : 16;
+    return product_floats(d, cols, kind) * 4 <= limit ? cols : 0;
 }
 
 // ------------------------------------------------------------------------------------------------ short runs
 // Thread (phase, group of V columns) has state rows phase, phase + phases, ...; a token's partial sums over the phases meet in
 // shared memory.  A single token's state rows (at most HELD a thread) are asked for ahead of the decays.
-constexpr int WALK_THREADS = 256;
 constexpr int HELD = 16;
 
 template <int V>
@@ -464,8 +510,8 @@ struct Cols {
     }
 };
 
-template <typename T, int V, bool HOLD>
-__global__ void __launch_bounds__(WALK_THREADS) channel_walk_kernel(const ChannelScan a, const float* __restrict__ gate, const float* __restrict__ norm,
+template <typename T, int V, bool HOLD, int WALK_THREADS>
+__global__ void __launch_bounds__(WALK_THREADS, 512 / WALK_THREADS) channel_walk_kernel(const ChannelScan a, const float* __restrict__ gate, const float* __restrict__ norm,
                                                                    float eps, T* __restrict__ out) {
     extern __shared__ __align__(16) float smem[];
     __shared__ float scratch[32];
@@ -584,14 +630,16 @@ int walk_launch(const ChannelScan& a, const float* norm, float eps, void* out, i
     const float* gate = a.v + (long)a.heads * a.dv;
     const bool vec = a.dv % 4 == 0 && a.state_len % 4 == 0 && a.stride % 4 == 0 && ((uintptr_t)a.v & 15) == 0 && ((uintptr_t)a.state & 15) == 0;
     const int V = vec ? 4 : 1, groups = (a.dv + V - 1) / V;
-    const int phases = groups < WALK_THREADS ? WALK_THREADS / groups : 1;
-    const bool hold = vec && longest == 1 && groups <= WALK_THREADS && (a.d + phases - 1) / phases <= HELD;
-    const size_t bytes = (3L * a.d + a.rank + a.dv + 4 + (long)WALK_THREADS * V) * sizeof(float);
+    // a single token's state in registers: with twice the threads where that is what it takes
+    const auto holds = [&](int threads) { return vec && longest == 1 && groups <= threads && (a.d + threads / groups - 1) / (threads / groups) <= HELD; };
+    const int threads = !holds(256) && holds(512) ? 512 : 256;
+    const size_t bytes = (3L * a.d + a.rank + a.dv + 4 + (long)threads * V) * sizeof(float);
     if (bytes > 47 * 1024) return KIRAI_ERR_UNSUPPORTED;
-    const dim3 grid(a.requests, a.heads), block(WALK_THREADS);
-    if (hold) return launch_pdl(channel_walk_kernel<T, 4, true>, grid, block, bytes, stream, 1u, a, gate, norm, eps, (T*)out);
-    if (vec) return launch_pdl(channel_walk_kernel<T, 4, false>, grid, block, bytes, stream, 1u, a, gate, norm, eps, (T*)out);
-    return launch_pdl(channel_walk_kernel<T, 1, false>, grid, block, bytes, stream, 1u, a, gate, norm, eps, (T*)out);
+    const dim3 grid(a.requests, a.heads), block(threads);
+    if (threads == 512) return launch_pdl(channel_walk_kernel<T, 4, true, 512>, grid, block, bytes, stream, 1u, a, gate, norm, eps, (T*)out);
+    if (holds(256)) return launch_pdl(channel_walk_kernel<T, 4, true, 256>, grid, block, bytes, stream, 1u, a, gate, norm, eps, (T*)out);
+    if (vec) return launch_pdl(channel_walk_kernel<T, 4, false, 256>, grid, block, bytes, stream, 1u, a, gate, norm, eps, (T*)out);
+    return launch_pdl(channel_walk_kernel<T, 1, false, 256>, grid, block, bytes, stream, 1u, a, gate, norm, eps, (T*)out);
 }
 
 }  // namespace
@@ -602,7 +650,7 @@ KIRAI_EXPORT int kirai_channel_chunks_fit(int d, int rank) {
     if (cudaGetDevice(&device) != cudaSuccess ||
         cudaDeviceGetAttribute(&limit, cudaDevAttrMaxSharedMemoryPerBlockOptin, device) != cudaSuccess)
         return 0;
-    return d > 0 && rank > 0 && product_floats(d, 16) * 4 <= limit && prepare_floats(d, rank) * 4 + 64 <= limit ? 1 : 0;
+    return d > 0 && rank > 0 && product_floats(d, 16, CHAIN) * 4 <= limit && prepare_floats(d, rank) * 4 + 64 <= limit ? 1 : 0;
 }
 
 // rows [T, 2 heads d + 2 heads dv + rank] (float32, row stride `stride`): q, k, v, the output gate's and the short decay rows.
@@ -638,8 +686,7 @@ KIRAI_EXPORT int kirai_channel_chunks(const float* rows, long stride, const floa
     if (status != 0) return status;
     if (units <= 0 || !tiles || !kept) return KIRAI_ERR_BAD_SIZE;
     a.out = o, a.tiles = tiles, a.kept = kept, a.share = share;
-    long bytes = 0;
-    a.cols = choose_cols((long)(share ? units : requests) * heads, d, dv, share != nullptr, &bytes);
+    a.cols = choose_cols((long)(share ? units : requests) * heads, d, dv, share != nullptr);
     if (a.cols <= 0) return KIRAI_ERR_UNSUPPORTED;
     const int runs = cols_pitch(a.cols) / 16, pieces = (dv + a.cols - 1) / a.cols;
     static long granted_prepare = 0, granted[3][5] = {};  // (one device a process)
@@ -650,14 +697,16 @@ KIRAI_EXPORT int kirai_channel_chunks(const float* rows, long stride, const floa
     if (status != 0) return status;
     if (!share) {
         auto chain = KIRAI_BY_RUNS(runs, channel_chain_kernel);
+        const long bytes = product_floats(d, a.cols, CHAIN) * 4;
         status = grant_shared(chain, bytes, &granted[0][runs]);
         return status != 0 ? status : launch_pdl(chain, dim3(requests, heads, pieces), dim3(THREADS), (size_t)bytes, stream, 1u, a);
     }
     auto own = KIRAI_BY_RUNS(runs, channel_share_kernel);
     auto out = KIRAI_BY_RUNS(runs, channel_out_kernel);
-    status = grant_shared(own, bytes, &granted[1][runs]);
+    const long own_bytes = product_floats(d, a.cols, SHARE) * 4, bytes = product_floats(d, a.cols, READ) * 4;
+    status = grant_shared(own, own_bytes, &granted[1][runs]);
     if (status == 0) status = grant_shared(out, bytes, &granted[2][runs]);
-    if (status == 0) status = launch_pdl(own, dim3(units, heads, pieces), dim3(THREADS), (size_t)bytes, stream, 1u, a);
+    if (status == 0) status = launch_pdl(own, dim3(units, heads, pieces), dim3(THREADS), (size_t)own_bytes, stream, 1u, a);
     if (status == 0)
         status = launch_pdl(channel_carry_kernel, dim3(requests, heads, (unsigned)(((long)d * dv + 255) / 256)), dim3(256), 0, stream, 1u, a);
     if (status == 0) status = launch_pdl(out, dim3(units, heads, pieces), dim3(THREADS), (size_t)bytes, stream, 1u, a);

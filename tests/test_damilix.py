@@ -422,7 +422,7 @@ FORMS = (dict(chain_limit=10 ** 9), dict(chain_limit=0), dict(walk_limit=10 ** 9
 @pytest.mark.gpu
 @pytest.mark.parametrize("spread", ["mild", "harsh"])
 @pytest.mark.parametrize("heads,dim,vdim,rank,tau", [(4, 16, 8, 16, 16.0), (3, 40, 20, 5, 2.0), (2, 128, 64, 16, 1.0), (1, 256, 80, 32, 4.0),
-                                                     (1, 3, 5, 1, 1.0), (2, 1, 300, 3, 8.0), (1, 20, 1100, 4, 3.0), (1, 500, 12, 8, 2.0)])
+                                                     (1, 3, 5, 1, 1.0), (2, 1, 300, 3, 8.0), (1, 20, 1100, 4, 3.0), (1, 500, 12, 8, 2.0), (2, 128, 256, 8, 16.0)])
 def test_runs_in_chunks_as_token_by_token(heads, dim, vdim, rank, tau, spread):
     """Six requests (a run that ends inside a piece of a chunk, on a chunk's edge, one behind it, several chunks, a single
     token) from states that are not zero: the three forms and a plain loop agree on the normed and gated outputs and on the
@@ -466,6 +466,19 @@ def test_runs_in_chunks_as_token_by_token(heads, dim, vdim, rank, tau, spread):
         for slot in range(8):
             want = states.get(slot, state0[slot].double().view(heads, dim, vdim))
             assert float((st[slot].cpu().double().view(heads, dim, vdim) - want).abs().max()) <= 3e-5 * max(1.0, float(want.abs().max())), (limits, slot)
+    # single tokens: every request's first row, from the same states (a state's rows in registers where they fit)
+    single = Session([StateNeed((L,), torch.float32)], torch.float32, page_size=4, num_pages=8, num_slots=8).batch([(f"r{i}", 1) for i in range(6)])
+    firsts = torch.tensor(starts[:-1])
+    st = state0.clone().cuda()
+    got = ops.channel_scan(rows[firsts].contiguous().cuda(), up.cuda(), bias.cuda(), tau, dim ** -0.5, st, single, heads, dim, vdim, norm.cuda(), 1e-3,
+                           torch.float32).cpu()
+    for r, first in enumerate(firsts.tolist()):
+        slot = int(single.slots[r])
+        one = slice(first, first + 1)
+        o, S = plain.linear_recurrence(q[one], k[one], v[one], log_a[one], state0[slot].double().view(heads, dim, vdim))
+        want = plain.unit_norm(o, norm[:vdim].double(), 1e-3).reshape(1, values) * plain.silu(gate[one])
+        assert float((got[r].double() - want).abs().max()) <= 1e-4 * max(1.0, float(want.abs().max())), ("single", r)
+        assert float((st[slot].cpu().double().view(heads, dim, vdim) - S).abs().max()) <= 3e-5 * max(1.0, float(S.abs().max())), ("single", slot)
     narrow = ops.channel_scan(rows.cuda(), up.cuda(), bias.cuda(), tau, dim ** -0.5, state0.clone().cuda(), batch, heads, dim, vdim, norm.cuda(),
                               1e-3, torch.bfloat16)
     assert narrow.dtype == torch.bfloat16
