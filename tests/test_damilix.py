@@ -350,6 +350,7 @@ LATENT_CASES = [  # kind, heads, dim, rot_dim, vdim, kv_rank, scale, base, scali
     ((HALVES, 3, 24, 16, 8, 40, 0.6, 500.0, (2.0, 16, 4.0, 0.5)), 64, 4),
     ((HALVES, 16, 8, 32, 16, 96, 0.5, 10000.0, None), 72, 8),
     ((NEIGHBOURS, 20, 8, 8, 4, 200, 0.6, 900.0, (3.0, 64, 4.0, 1.0)), 56, 16),
+    ((HALVES, 2, 12, 40, 16, 260, 0.5, 2000.0, None), 64, 8),  # a cached row wider than the tensor-core kernels take
 ]
 
 
