@@ -673,6 +673,14 @@ def plain_reference(config, weights, tokens):
     return logits, bounds, sure.numpy()
 
 
+def long_reference(tiny, tokens):
+    """``plain_reference`` of a sequence, worked out once for both precisions."""
+    known = tiny.setdefault("long", {})
+    if tuple(tokens) not in known:
+        known[tuple(tokens)] = plain_reference(tiny["config"], tiny["weights"], tokens)
+    return known[tuple(tokens)]
+
+
 def check(dtype, got, reference, rows, what):
     logits, bounds, sure = reference
     rows = np.asarray(list(rows))
@@ -755,7 +763,7 @@ def test_a_long_prompt_whole_and_in_portions(tiny, dtype, tmp_path):
 
     toks = random_tokens(330, tiny["raw"]["vocab"], 77)
     other = tiny["sequences"]["d"]
-    reference = plain_reference(tiny["config"], tiny["weights"], toks)
+    reference = long_reference(tiny, toks)
     rows = [0, 1, 15, 16, 63, 64, 65, 127, 128, 200, 255, 256, 257, 300, 328, 329]
     replay = Replay(tiny["folder"], dtype, str(tmp_path / "out"), max_tokens=512, page_size=tiny["page"])
     got = replay.step([("long", toks, rows), ("d", other, [len(other) - 1])], end=["long", "d"])
@@ -825,7 +833,7 @@ def test_first_tokens_and_long_decoding(tiny, dtype, tmp_path):
     from replay_client import Replay
 
     toks = random_tokens(330, tiny["raw"]["vocab"], 17)
-    reference = plain_reference(tiny["config"], tiny["weights"], toks)
+    reference = long_reference(tiny, toks)
     replay = Replay(tiny["folder"], dtype, str(tmp_path / "out"), max_tokens=352, page_size=tiny["page"])
     for i, token in enumerate(toks):
         got = replay.step([("long", [token], [0])])
